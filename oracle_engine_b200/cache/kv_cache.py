@@ -7,8 +7,8 @@ owns its storage (per declared tensor [entries, pages, *outer, PAGE, inner]; for
 the one tensor "kv" [entries, pages, 2 (K,V), kv_heads, PAGE, head_dim]), its page pool
 and, for each slot, one page table shared by the group's entries (they all hold the same
 positions).  A "full" group keeps every position of a sequence; a "window" group gives a
-page back as soon as all of its positions lie before the window of the next query, so its
-pool can be smaller.  Slots and pages return to their pools when a sequence ends and are
+page back as soon as all of its positions lie before the window of the next query, a "chunk"
+group as soon as they lie in chunks the next query has left, so their pools can be smaller.  Slots and pages return to their pools when a sequence ends and are
 handed out again; nothing is cleared, since a position is readable only after it has
 been written (each sequence's length bounds every read).
 
@@ -56,7 +56,7 @@ class CacheGroup:
         self.entries = entries
         self.pool = PagePool(n_pages)
         self.tables = np.full((n_slots, max_pages_per_seq), -1, dtype=np.int32)
-        # per slot: pages [lo, hi) are mapped (lo > 0 only in window groups)
+        # per slot: pages [lo, hi) are mapped (lo > 0 only in window and chunk groups)
         self.lo = np.zeros(n_slots, dtype=np.int64)
         self.hi = np.zeros(n_slots, dtype=np.int64)
         self.storage: dict | None = None        # tensor name -> [entries, pages, *outer, PAGE, inner]
@@ -96,10 +96,10 @@ class KVCache:
         for e, need in enumerate(needs):
             if need is None:
                 continue
-            if need.kind not in ("full", "window"):
+            if need.kind not in ("full", "window", "chunk"):
                 raise ValueError(f"entry {e}: unknown cache kind {need.kind!r}")
-            if need.kind == "window" and need.window < 1:
-                raise ValueError(f"entry {e}: a window cache needs window >= 1")
+            if need.kind != "full" and min([need.window] + [n for _, n in need.also]) < 1:
+                raise ValueError(f"entry {e}: a {need.kind} cache needs a size >= 1")
             names = [name for name, _ in need.tensors]
             if not names or len(set(names)) != len(names):
                 raise ValueError(f"entry {e}: a cache need declares at least one tensor, each name once")
@@ -108,7 +108,7 @@ class KVCache:
             by_need.setdefault(need, []).append(e)
         for gi, (need, entries) in enumerate(by_need.items()):
             pages = n_pages
-            if need.kind == "window" and window_pool_tokens is not None:
+            if need.kind != "full" and window_pool_tokens is not None:
                 pages = min(n_pages, max(1, window_pool_tokens // PAGE))
             g = CacheGroup(gi, need, entries, pages, self.n_slots, self.max_pages_per_seq)
             self.groups.append(g)
@@ -144,7 +144,7 @@ class KVCache:
     # ------------------------------------------------------------------ pages
     def reserve(self, slot: int, new_len: int) -> bool:
         """Makes positions [length, new_len) of `slot` writable in every group (and, in
-        window groups, releases pages no query of this step can reach).  Returns True if
+        window and chunk groups, releases pages no query of this step can reach).  Returns True if
         any page table changed.  Raises CacheFull before changing anything it cannot
         finish for this slot."""
         if not self.slots.is_held(slot):
@@ -154,8 +154,8 @@ class KVCache:
             raise CacheFull(f"sequence would reach {new_len} tokens; the cache allows {self.max_seq_len}")
         need_hi = pages_for(new_len)
         for g in self.groups:                       # the common case: every page is there already
-            if need_hi > g.hi[slot] or (g.need.kind == "window"
-                                        and max(0, cur - g.need.window + 1) // PAGE > g.lo[slot]):
+            if need_hi > g.hi[slot] or (g.need.kind != "full"
+                                        and g.need.first_position(cur) // PAGE > g.lo[slot]):
                 break
         else:
             return False
@@ -163,8 +163,8 @@ class KVCache:
         first_needed_page = {}
         for g in self.groups:
             lo_page = 0
-            if g.need.kind == "window":
-                lo_page = max(0, cur - g.need.window + 1) // PAGE     # oldest key the first new query reads
+            if g.need.kind != "full":
+                lo_page = g.need.first_position(cur) // PAGE          # oldest key the first new query reads
             first_needed_page[g.index] = lo_page
             row = g.tables[slot]
             releasable = int(((row[:lo_page] >= 0).sum()))

@@ -9,7 +9,8 @@
 // is a multiple of 2 up to 256).
 // Reference: core/model.cpp:411-435 (decode) and :605-626 (prefill): query head h reads
 // KV head h / (H/KVH); s_t = (q.k_t)/sqrt(hd) for keys t <= pos; softmax; o = sum s_t v_t.
-// `window` > 0 restricts the keys to pos-window < t <= pos (0 = all keys).
+// `window` > 0 restricts the keys to pos-window < t <= pos, `window` < 0 to those of the query's own chunk of -window
+// positions (0 = all keys; common.cuh: oe_first_key).
 // `sink` != 0 adds one to the softmax's denominator: a key of score 0 that has no value
 // (the running maximum starts at 0 and the running sum at 1).
 #include "common.cuh"
@@ -40,7 +41,7 @@ attn_paged_kernel(T* out, const T* q, int q_stride,
         return;
     }
     const int pos = tok_pos[t];
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = oe_first_key(pos, window);
     const int kvh = h / (H / KVH);
     const int* trow = tables + (size_t)b * max_pages;
     const T* qr = q + (size_t)t * q_stride + (size_t)h * hd;

@@ -9,7 +9,7 @@
 // in shared memory with cp.async, double buffered.  S = Q K^T and O += P V run on
 // mma.sync m16n8k16 (bf16 in, float32 accumulate) with ldmatrix fragments; the softmax is
 // online, in float32 (running maximum and sum per row).  Causal mask: key <= the row's
-// absolute position; window > 0 keeps only the last `window` keys.
+// absolute position; window > 0 keeps only the last `window` keys, window < 0 those of the row's own chunk of -window positions.
 // For decoded tokens the page range of a sequence is split over `n_splits` CTAs; each
 // writes an unnormalised partial (o, m, l) and attn_merge_kernel combines them in split
 // order.
@@ -127,7 +127,7 @@ attn_mma_kernel(const AttnArgs a) {
     const int t0 = q_tile * tpt;
     const int nt = min(tpt, qlen - t0);
     const int pos_lo = start + t0, pos_hi = start + t0 + nt - 1;
-    const int key_lo = a.window > 0 ? max(0, pos_lo - a.window + 1) : 0;
+    const int key_lo = oe_first_key(pos_lo, a.window);
     int j_lo = key_lo / BN, j_hi = pos_hi / BN;
     if (a.n_splits > 1) {
         const int per = (j_hi - j_lo + a.n_splits) / a.n_splits;
@@ -149,7 +149,7 @@ attn_mma_kernel(const AttnArgs a) {
     const int row0 = warp * 16 + gid;                   // this thread's rows: row0 and row0 + 8
     const long long packed0 = a.cu_q[b] + t0;
 
-    int tok[2], pos[2], head[2];
+    int tok[2], pos[2], first[2], head[2];
     bool valid[2];
 #pragma unroll
     for (int i = 0; i < 2; i++) {
@@ -158,6 +158,7 @@ attn_mma_kernel(const AttnArgs a) {
         head[i] = kvh * G + r % G;
         valid[i] = tok[i] < nt;
         pos[i] = start + t0 + tok[i];
+        first[i] = oe_first_key(pos[i], a.window);
     }
 
     // Q fragments (A operand), kept in registers for the whole kernel
@@ -277,7 +278,7 @@ attn_mma_kernel(const AttnArgs a) {
             for (int e = 0; e < 4; e++) {
                 const int i = e >> 1;
                 const int key = j * BN + n * 8 + tig * 2 + (e & 1);
-                const bool ok = valid[i] && key <= pos[i] && (a.window <= 0 || key > pos[i] - a.window);
+                const bool ok = valid[i] && key <= pos[i] && key >= first[i];
                 const float s = ok ? sacc[n][e] * a.scale_log2 : -INFINITY;
                 sacc[n][e] = s;
                 rmax[i] = fmaxf(rmax[i], s);
@@ -496,7 +497,7 @@ attn_decode_warps_kernel(const AttnArgs a) {
         return;
     }
     const int pos = a.seq_start[b];                          // the new token's position
-    const int key_lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const int key_lo = oe_first_key(pos, a.window);
     const int hp_lo = key_lo / TB, hp_hi = pos / TB;
     const int* trow = a.tables + (size_t)b * a.max_pages;
     uint8_t* mine = smem + (size_t)warp * WARP_BYTES;

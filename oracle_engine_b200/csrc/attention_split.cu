@@ -8,7 +8,7 @@
 //                         [pages, G, PAGE, dv].
 //   attn_split            one warp per (token, query head): s_j = scale q.k_j, then s_j <- cap tanh(s_j / cap)
 //                         when cap > 0, for the keys pos - window < j <= pos (all keys up to pos when window
-//                         is 0); online softmax in float32 over chunks of 32 keys at absolute multiples of 32,
+//                         is 0, those of the query's own chunk of -window positions when it is negative); online softmax in float32 over chunks of 32 keys at absolute multiples of 32,
 //                         so a token's result does not depend on how the step was cut or batched.  The
 //                         32-bit path's attention, and the bfloat16 path's for head sizes that the tensor-core
 //                         kernel (attention_split_mma.cu) does not take.  `sinks` (null, or one float32 per query
@@ -100,7 +100,7 @@ attn_split_kernel(T* out, const T* q, long long q_stride, const T* kcache, const
         return;
     }
     const int pos = tok_pos[t];
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = oe_first_key(pos, window);
     const int g = h / (H / G);
     const int* trow = tables + (size_t)b * max_pages;
     const T* qr = q + (size_t)t * q_stride + (size_t)h * dk;

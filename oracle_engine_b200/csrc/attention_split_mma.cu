@@ -9,7 +9,7 @@
 // contiguous and are staged in shared memory with cp.async, double buffered.  S = Q K^T and O += P V run on
 // mma.sync m16n8k16 (bf16 in, float32 accumulate) with ldmatrix fragments.  Scores are float32: s = scale q.k,
 // then s <- cap tanh(s / cap) when cap > 0 (tanh as 1 - 2 / (exp(2x) + 1)); the softmax is online, in float32.
-// Mask: pos - window < key <= pos (window 0: every key up to pos).  Only the pages that hold a tile's visible
+// Mask: pos - window < key <= pos (window 0: every key up to pos; window < 0: the query's own chunk of -window positions).  Only the pages that hold a tile's visible
 // keys are read, so a windowed layer's cost does not grow with the context.
 // A step of single tokens may split a sequence's pages over `n_splits` CTAs (grid x): each writes its unnormalised
 // sums, maximum and denominator as float32, and attn_split_merge_kernel puts them together in split order.
@@ -111,7 +111,7 @@ attn_split_mma_kernel(const Args a) {
     if (t0 >= qlen) return;
     const int nt = min(tpt, qlen - t0);
     const int pos_lo = start + t0, pos_hi = start + t0 + nt - 1;
-    const int key_lo = a.window > 0 ? max(0, pos_lo - a.window + 1) : 0;
+    const int key_lo = oe_first_key(pos_lo, a.window);
     int j_lo = key_lo / BN, j_hi = pos_hi / BN;
     if (a.n_splits > 1) {
         const int per = (j_hi - j_lo + a.n_splits) / a.n_splits;
@@ -128,7 +128,7 @@ attn_split_mma_kernel(const Args a) {
     if (n_blocks > 0) load_page(smem, smem + K_TILE, a, trow[j_lo], kvh);
     cp_async_commit();
 
-    int tok[2], pos[2], head[2];
+    int tok[2], pos[2], first[2], head[2];
     bool valid[2];
 #pragma unroll
     for (int i = 0; i < 2; i++) {
@@ -137,6 +137,7 @@ attn_split_mma_kernel(const Args a) {
         head[i] = kvh * G + r % G;
         valid[i] = tok[i] < nt;
         pos[i] = start + t0 + tok[i];
+        first[i] = oe_first_key(pos[i], a.window);
     }
     uint32_t qf[KS][4];
 #pragma unroll
@@ -204,7 +205,7 @@ attn_split_mma_kernel(const Args a) {
             for (int e = 0; e < 4; e++) {
                 const int i = e >> 1;
                 const int key = j * BN + n * 8 + tig * 2 + (e & 1);
-                const bool ok = valid[i] && key <= pos[i] && (a.window <= 0 || key > pos[i] - a.window);
+                const bool ok = valid[i] && key <= pos[i] && key >= first[i];
                 float s;
                 if (a.cap > 0.f) {
                     const float ex = __expf(sacc[n][e] * two_over_cap);              // exp(2 s / cap)

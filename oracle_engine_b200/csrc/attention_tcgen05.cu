@@ -7,7 +7,7 @@
 //   S = Q K^T      tcgen05.mma M=128 N=64 K=head_dim, Q and K tiles K-major in 128B-swizzled
 //                  shared memory (TMA), S float32 in tensor memory (two buffers);
 //   softmax        128 threads, one row each: tcgen05.ld of the row's 64 scores, causal /
-//                  window mask, maximum and sum in float32 (no shuffles: a thread holds its
+//                  window or chunk mask, maximum and sum in float32 (no shuffles: a thread holds its
 //                  whole row), P = exp2(s * scale - m) rounded to bf16 and stored back into
 //                  the first half of the same tensor-memory columns (tcgen05.st);
 //   O += P V       tcgen05.mma M=128 N=head_dim K=64, P as the A operand from tensor memory,
@@ -262,7 +262,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         t0 = q_tile * tpt;
         nt = min(tpt, qlen - t0);
         const int pos_lo = start + t0, pos_hi = start + t0 + nt - 1;
-        const int key_lo = a.window > 0 ? max(0, pos_lo - a.window + 1) : 0;
+        const int key_lo = oe_first_key(pos_lo, a.window);
         j_lo = key_lo / BN;
         n_blocks = pos_hi / BN - j_lo + 1;
         packed0 = a.cu_q[b] + t0;
@@ -368,6 +368,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         const int tok = r / G, head = kvh * G + r % G;
         const bool valid = active && tok < nt;
         const int pos = start + t0 + tok;
+        const int first = oe_first_key(pos, a.window);       // the first key the row sees
         // m_run in units of the scaled scores (log2).  With a sink the maximum starts at the sink's score, 0,
         // and the sum holds the sink's weight 2^(0 - m_run) from the first block on.
         float m_run = a.sink ? 0.f : -INFINITY, l_run = 0.f;
@@ -387,14 +388,14 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             // 42 tokens x 3 heads, and a prompt's last tile fewer) take the unmasked path with whatever
             // their scores are, since every row's maximum, sum and output are that row's own and those
             // rows are never stored; left to each row, one such row made its warp run both paths.
-            const bool needs_mask = valid && !(key0 + BN - 1 <= pos && (a.window <= 0 || key0 > pos - a.window));
+            const bool needs_mask = valid && !(key0 + BN - 1 <= pos && key0 >= first);
             if (!__any_sync(0xffffffffu, needs_mask)) {
 #pragma unroll
                 for (int c = 0; c < BN; c++) mx4[c & 3] = fmaxf(mx4[c & 3], s[c]);
             } else {
                 // keys key0 + c with lo <= c <= hi stay (one unsigned comparison per score)
                 const int hi = valid ? min(pos - key0, BN - 1) : -1;
-                const int lo = a.window > 0 ? max(pos - a.window + 1 - key0, 0) : 0;
+                const int lo = max(first - key0, 0);
                 const unsigned span = hi >= lo ? (unsigned)(hi - lo) : 0u;
                 const bool any = hi >= lo;
 #pragma unroll

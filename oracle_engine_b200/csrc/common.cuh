@@ -99,6 +99,15 @@ static inline int oe_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, siz
     return oe_launch_ex(true, kernel, grid, block, smem, st, args...);
 }
 
+// The first key a query at position `pos` sees; its last one is its own.  `span` is what the attention entry points
+// call `window`: 0, every key of the sequence; n > 0, the last n keys (pos - n < key); -n < 0, the keys of the query's own
+// chunk, positions being cut into chunks of n from position 0 of the sequence on (key / n == pos / n).
+__device__ __forceinline__ int oe_first_key(int pos, int span) {
+    if (span > 0) return pos >= span ? pos - span + 1 : 0;
+    if (span < 0) return pos - pos % -span;
+    return 0;
+}
+
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(bf16 v) { return __bfloat162float(v); }
 
@@ -116,6 +125,9 @@ __device__ __forceinline__ float warp_max(float v) {
     for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
     return v;
 }
+
+// z times the normal distribution function: the exact gelu.
+__device__ __forceinline__ float oe_gelu(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
 // Sum over a block in a fixed order (warp shuffles, then warp 0 over the warp totals);
 // every thread gets the result.  `red` holds 32 floats of shared memory.

@@ -149,6 +149,107 @@ rmsnorm_rows_kernel(T* y, const float* x, const float* __restrict__ w, int rows,
 }
 
 // ---------------------------------------------------------------------------------------
+// y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b: the mean first, then the mean of the squared deviations
+// from it, both float32 sums in an order that D and the launch form fix.
+// ---------------------------------------------------------------------------------------
+template <typename T>
+__global__ void layernorm_kernel(T* y, const float* x, const float* __restrict__ w, const float* __restrict__ b, int D,
+                                 float eps) {
+    __shared__ float red[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const float* xr = x + (size_t)blockIdx.x * D;
+    T* yr = y + (size_t)blockIdx.x * D;
+    float sum = 0.f, sq = 0.f;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) sum += xr[d];
+    const float mean = block_sum(sum, red) / (float)D;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) { const float v = xr[d] - mean; sq = fmaf(v, v, sq); }
+    const float s = 1.f / sqrtf(block_sum(sq, red) / (float)D + eps);
+    for (int d = threadIdx.x; d < D; d += blockDim.x) yr[d] = from_f32<T>(fmaf((xr[d] - mean) * s, w[d], b[d]));
+}
+
+__device__ __forceinline__ float sum4(const float4& v) { return (v.x + v.y) + (v.z + v.w); }
+__device__ __forceinline__ float dev4(const float4& v, float mean) {
+    const float a = v.x - mean, b = v.y - mean, c = v.z - mean, d = v.w - mean;
+    return fmaf(a, a, b * b) + fmaf(c, c, d * d);
+}
+template <typename T>
+__device__ __forceinline__ void layernorm_store(T* p, const float4& v, float mean, float s, const float4& g, const float4& o) {
+    Out4<T>::store(p, fmaf((v.x - mean) * s, g.x, o.x), fmaf((v.y - mean) * s, g.y, o.y), fmaf((v.z - mean) * s, g.z, o.z),
+                   fmaf((v.w - mean) * s, g.w, o.w));
+}
+
+// A block per row, 16-byte pieces, up to 16 NT columns of the row in registers: both passes read them there.
+template <typename T, int NT>
+__global__ void __launch_bounds__(NT)
+layernorm_vec_kernel(T* y, const float* x, const float* __restrict__ w, const float* __restrict__ b, int D, float eps) {
+    __shared__ float red[32];
+    constexpr int KEEP = 4;
+    pdl_launch_dependents();
+    pdl_wait();
+    const float4* xr = (const float4*)(x + (size_t)blockIdx.x * D);
+    const float4 *wr = (const float4*)w, *br = (const float4*)b;
+    T* yr = y + (size_t)blockIdx.x * D;
+    const int n4 = D / 4;
+    float4 keep[KEEP];
+    float sum = 0.f, sq = 0.f;
+#pragma unroll
+    for (int j = 0; j < KEEP; j++) {
+        const int i = threadIdx.x + j * NT;
+        keep[j] = i < n4 ? xr[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        sum += sum4(keep[j]);
+    }
+    for (int i = threadIdx.x + KEEP * NT; i < n4; i += NT) sum += sum4(xr[i]);
+    const float mean = block_sum(sum, red) / (float)D;
+#pragma unroll
+    for (int j = 0; j < KEEP; j++)
+        if (threadIdx.x + j * NT < n4) sq += dev4(keep[j], mean);
+    for (int i = threadIdx.x + KEEP * NT; i < n4; i += NT) sq += dev4(xr[i], mean);
+    const float s = 1.f / sqrtf(block_sum(sq, red) / (float)D + eps);
+#pragma unroll
+    for (int j = 0; j < KEEP; j++) {
+        const int i = threadIdx.x + j * NT;
+        if (i < n4) layernorm_store(yr + 4 * i, keep[j], mean, s, wr[i], br[i]);
+    }
+    for (int i = threadIdx.x + KEEP * NT; i < n4; i += NT) layernorm_store(yr + 4 * i, xr[i], mean, s, wr[i], br[i]);
+}
+
+// Many rows: a warp per row, the row (KEEP x 32 float4) in registers, as rmsnorm_rows_kernel.
+template <typename T, int KEEP>
+__global__ void __launch_bounds__(256)
+layernorm_rows_kernel(T* y, const float* x, const float* __restrict__ w, const float* __restrict__ b, int rows, int D,
+                      float eps) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (r >= rows) return;
+    const float4* xr = (const float4*)(x + (size_t)r * D);
+    const float4 *wr = (const float4*)w, *br = (const float4*)b;
+    T* yr = y + (size_t)r * D;
+    const int n4 = D / 4;
+    float4 keep[KEEP];
+    float sum = 0.f, sq = 0.f;
+#pragma unroll
+    for (int j = 0; j < KEEP; j++) {
+        const int i = lane + j * 32;
+        keep[j] = i < n4 ? xr[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; j++) sum += sum4(keep[j]);
+    const float mean = warp_sum(sum) / (float)D;
+#pragma unroll
+    for (int j = 0; j < KEEP; j++)
+        if (lane + j * 32 < n4) sq += dev4(keep[j], mean);
+    const float s = 1.f / sqrtf(warp_sum(sq) / (float)D + eps);
+#pragma unroll
+    for (int j = 0; j < KEEP; j++) {
+        const int i = lane + j * 32;
+        if (i < n4) layernorm_store(yr + 4 * i, keep[j], mean, s, wr[i], br[i]);
+    }
+}
+
+// ---------------------------------------------------------------------------------------
 // Rotary encoding of q and k (rotate-half pairs (i, i+hd/2)) at each token's absolute
 // position, from a float32 cos/sin table [max_pos, hd/2]; q is rotated in place, rotated
 // k and v go to the token's row of the paged cache.
@@ -473,6 +574,27 @@ int oe_rmsnorm_bf16(bf16* y, const float* x, const float* w, int rows, int D, fl
     }
     const int launch_rc = oe_launch(rmsnorm_kernel<bf16>, dim3(rows), dim3(256), 0, st, y, x, w, D, eps);
     return launch_rc;
+}
+
+int oe_layernorm_f32(float* y, const float* x, const float* w, const float* b, int rows, int D, float eps, cudaStream_t st) {
+    if (rows <= 0) return 0;
+    if (D % 4 == 0 && !(((uintptr_t)y | (uintptr_t)x | (uintptr_t)w | (uintptr_t)b) & 15))
+        return oe_launch(layernorm_vec_kernel<float, 256>, dim3(rows), dim3(256), 0, st, y, x, w, b, D, eps);
+    return oe_launch(layernorm_kernel<float>, dim3(rows), dim3(256), 0, st, y, x, w, b, D, eps);
+}
+int oe_layernorm_bf16(bf16* y, const float* x, const float* w, const float* b, int rows, int D, float eps, cudaStream_t st) {
+    if (rows <= 0) return 0;
+    if (D % 4 == 0 && !(((uintptr_t)x | (uintptr_t)w | (uintptr_t)b) & 15) && !((uintptr_t)y & 7)) {
+        if (rows >= OE_RMSNORM_ROWS_MIN && D <= 4096) {
+            const dim3 grid((rows + 7) / 8);
+            if (D <= 1024) return oe_launch(layernorm_rows_kernel<bf16, 8>, grid, dim3(256), 0, st, y, x, w, b, rows, D, eps);
+            if (D <= 2048) return oe_launch(layernorm_rows_kernel<bf16, 16>, grid, dim3(256), 0, st, y, x, w, b, rows, D, eps);
+            if (D <= 3072) return oe_launch(layernorm_rows_kernel<bf16, 24>, grid, dim3(256), 0, st, y, x, w, b, rows, D, eps);
+            return oe_launch(layernorm_rows_kernel<bf16, 32>, grid, dim3(256), 0, st, y, x, w, b, rows, D, eps);
+        }
+        return oe_launch(layernorm_vec_kernel<bf16, 512>, dim3(rows), dim3(512), 0, st, y, x, w, b, D, eps);
+    }
+    return oe_launch(layernorm_kernel<bf16>, dim3(rows), dim3(256), 0, st, y, x, w, b, D, eps);
 }
 
 int oe_rope_kv_write_f32(float* qkv, int row_stride, const float* cos_tab, const float* sin_tab,

@@ -9,18 +9,23 @@
 //                   a gate; z then holds no column for it).  mode 1: the weight of a chosen expert is the sigmoid
 //                   of its own logit, not renormalised (the choice is by the same order).  With `bias` (one float32
 //                   per expert, mode 1 only) the choice is by sigmoid(z) + bias and the weight stays sigmoid(z).
+//                   mode 2: the scores are the softmax over ALL experts, the weights the chosen scores over (their sum
+//                   + 1e-20).  n_groups > 0: the experts stand in n_groups equal runs, a run's score is its best
+//                   expert's, and only experts of the `keep` best runs can be chosen.
 //   moe_dense_act   gu [T, 2 F] holds, for F = E ff + shared_ff columns, the gate rows and, F columns further, the
 //                   up rows of all experts (expert e owns columns e ff .. (e + 1) ff - 1, the shared expert the last
 //                   shared_ff).  a[t, c] = silu(gate) * up * dense[t, expert of c]: the experts a token did not
 //                   choose contribute zeros to the one product with all down matrices that follows.  scale_input:
 //                   the weight multiplies the expert's input instead of its output, a = silu(w gate) * (w up).
+//   moe_dense_relu2   the same for experts without a gate, in place: u[t, c] = max(u[t, c], 0)^2 * dense[t, c / ff].
 #include "common.cuh"
 
 namespace {
 
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* z, long long ldz, int E, int top, int has_gate, int mode, int* idx, float* wt, float* dense,
-                 const int* __restrict__ tok_seq, int n_tokens, const float* __restrict__ bias) {
+                 const int* __restrict__ tok_seq, int n_tokens, const float* __restrict__ bias, int n_groups, int keep) {
+    __shared__ unsigned kept_runs[4][32];
     pdl_launch_dependents();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -38,6 +43,34 @@ moe_route_kernel(const float* z, long long ldz, int E, int top, int has_gate, in
     }
     __syncwarp();
     const float* zr = z + (size_t)t * ldz;
+    // what the choice goes by: a logit (its order is the softmax's), or sigmoid + bias
+    auto score = [&](int e) { return bias ? 1.f / (1.f + expf(-zr[e])) + bias[e] : zr[e]; };
+    unsigned* kept = kept_runs[warp];        // bit g: run g stays in the race
+    const int per_run = n_groups > 0 ? E / n_groups : E;
+    if (n_groups > 0) {
+        kept[lane] = 0u;
+        __syncwarp();
+        for (int j = 0; j < keep; j++) {
+            float best = -INFINITY;
+            int bg = 0x7fffffff;
+            for (int g = lane; g < n_groups; g += 32) {
+                if (kept[g >> 5] >> (g & 31) & 1u) continue;
+                float v = -INFINITY;
+                for (int e = g * per_run; e < (g + 1) * per_run; e++) v = fmaxf(v, score(e));
+                if (v > best || (v == best && g < bg)) { best = v; bg = g; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+                const int og = __shfl_xor_sync(0xffffffffu, bg, o);
+                if (ov > best || (ov == best && og < bg)) { best = ov; bg = og; }
+            }
+            if (bg == 0x7fffffff) break;
+            __syncwarp();
+            if (lane == 0) kept[bg >> 5] |= 1u << (bg & 31);
+            __syncwarp();
+        }
+    }
     unsigned taken = 0;                      // bit i: this lane's element lane + 32 i is chosen already
     float zmax = 0.f, sum = 0.f;
     // pass 1: choose; the first chosen logit is the largest and anchors the exponentials
@@ -46,7 +79,8 @@ moe_route_kernel(const float* z, long long ldz, int E, int top, int has_gate, in
         int bi = 0x7fffffff;
         for (int i = 0, e = lane; e < E; e += 32, i++) {
             if (taken >> i & 1u) continue;
-            const float v = bias ? 1.f / (1.f + expf(-zr[e])) + bias[e] : zr[e];
+            if (n_groups > 0 && !(kept[(e / per_run) >> 5] >> ((e / per_run) & 31) & 1u)) continue;
+            const float v = score(e);
             if (v > best || (v == best && e < bi)) { best = v; bi = e; }
         }
 #pragma unroll
@@ -67,7 +101,15 @@ moe_route_kernel(const float* z, long long ldz, int E, int top, int has_gate, in
         }
     }
     __syncwarp();
-    const float inv = mode == 1 ? 1.f : 1.f / sum;
+    float inv = mode == 1 ? 1.f : 1.f / sum;
+    if (mode == 2) {
+        // zmax is the largest logit of all: the best run holds it.  With Z = sum_all exp(z - zmax) a score is
+        // p / Z, and p / Z / (sum / Z + 1e-20) is the weight.
+        float total = 0.f;
+        for (int e = lane; e < E; e += 32) total += expf(zr[e] - zmax);
+        total = warp_sum(total);
+        inv = 1.f / total / (sum / total + 1e-20f);
+    }
     for (int i = 0, e = lane; e < E; e += 32, i++)
         if (taken >> i & 1u) drow[e] *= inv;
     if (wt) for (int j = lane; j < top; j += 32) wt[(size_t)t * top + j] *= inv;
@@ -124,6 +166,49 @@ moe_dense_act_kernel(T* a, const T* gu, const float* dense, int n_tokens, int F,
     }
 }
 
+// In place; a thread takes 8 consecutive columns (16 bytes of bfloat16) or one; the columns of an expert the token did
+// not choose become zero unread.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+moe_dense_relu2_kernel(T* u, const float* dense, int n_tokens, int F, int ff, int W) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int per_row = F / V;
+    const size_t total = (size_t)n_tokens * per_row;
+    for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = e / per_row;
+        const int c = (int)(e % per_row) * V;
+        const float w = dense[t * W + c / ff];
+        T v[V];
+        if (w != 0.f) {
+            if (V == 8) *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(u + t * F + c);
+            else v[0] = u[t * F + c];
+#pragma unroll
+            for (int i = 0; i < V; i++) {
+                const float r = fmaxf(to_f32(v[i]), 0.f);
+                v[i] = from_f32<T>(r * r * w);
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < V; i++) v[i] = from_f32<T>(0.f);
+        }
+        if (V == 8) *reinterpret_cast<uint4*>(u + t * F + c) = *reinterpret_cast<uint4*>(v);
+        else u[t * F + c] = v[0];
+    }
+}
+
+template <typename T>
+int launch_relu2(T* u, const float* dense, int n_tokens, int F, int ff, int W, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
+    if (F < 1 || ff < 1 || F % ff || W < F / ff) return OE_ERR_UNSUPPORTED;
+    const bool vec = sizeof(T) == 2 && ff % 8 == 0 && !((uintptr_t)u & 15);
+    const size_t total = (size_t)n_tokens * (vec ? F / 8 : F);
+    size_t blocks = (total + 255) / 256;
+    if (blocks > 148 * 16) blocks = 148 * 16;
+    if (vec) return oe_launch(moe_dense_relu2_kernel<T, 8>, dim3((unsigned)blocks), dim3(256), 0, st, u, dense, n_tokens, F, ff, W);
+    return oe_launch(moe_dense_relu2_kernel<T, 1>, dim3((unsigned)blocks), dim3(256), 0, st, u, dense, n_tokens, F, ff, W);
+}
+
 template <typename T>
 int launch_act(T* a, const T* gu, const float* dense, int n_tokens, int F, int E, int ff, int W, int scale_input,
                int act, float limit, cudaStream_t st) {
@@ -144,11 +229,18 @@ int launch_act(T* a, const T* gu, const float* dense, int n_tokens, int F, int E
 extern "C" {
 
 int oe_moe_route(const float* z, long long ldz, int E, int top, int has_gate, int mode, int* idx, float* wt, float* dense,
-                 const int* tok_seq, int n_tokens, const float* bias, cudaStream_t st) {
+                 const int* tok_seq, int n_tokens, const float* bias, int n_groups, int keep, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
-    if (E < 1 || E > 1024 || top < 1 || (bias != nullptr && mode != 1)) return OE_ERR_UNSUPPORTED;
+    if (E < 1 || E > 1024 || top < 1 || mode < 0 || mode > 2 || (bias != nullptr && mode != 1)) return OE_ERR_UNSUPPORTED;
+    if (n_groups < 0 || (n_groups > 0 && (E % n_groups || keep < 1 || keep > n_groups))) return OE_ERR_UNSUPPORTED;
     return oe_launch(moe_route_kernel, dim3((n_tokens + 3) / 4), dim3(128), 0, st, z, ldz, E, top, has_gate, mode, idx, wt, dense,
-                     tok_seq, n_tokens, bias);
+                     tok_seq, n_tokens, bias, n_groups, keep);
+}
+int oe_moe_dense_relu2_f32(float* u, const float* dense, int n_tokens, int F, int ff, int W, cudaStream_t st) {
+    return launch_relu2<float>(u, dense, n_tokens, F, ff, W, st);
+}
+int oe_moe_dense_relu2_bf16(bf16* u, const float* dense, int n_tokens, int F, int ff, int W, cudaStream_t st) {
+    return launch_relu2<bf16>(u, dense, n_tokens, F, ff, W, st);
 }
 int oe_moe_dense_act_f32(float* a, const float* gu, const float* dense, int n_tokens, int F, int E, int ff, int W,
                          int scale_input, int act, float limit, cudaStream_t st) {

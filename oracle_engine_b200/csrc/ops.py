@@ -35,6 +35,7 @@ _SIGNATURES = {
     "elementwise": {
         "oe_embed_gather": [_P, _P, _P, _I, _I, _I, _P, _P],
         "oe_rmsnorm": [_P, _P, _P, _I, _I, _F, _P],
+        "oe_layernorm": [_P, _P, _P, _P, _I, _I, _F, _P],
         "oe_rope_kv_write": [_P, _I, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
         "oe_swiglu": [_P, _P, _I, _I, _P],
         "oe_gather_rows_f32": [_P, _P, _P, _I, _I, _P],
@@ -49,6 +50,7 @@ _SIGNATURES = {
         "oe_cast_rows_bf16": [_P, _P, _L, _P],
         "oe_rmsnorm_add": [_P, _P, _P, _I, _I, _F, _F, _I, _P, _P],
         "oe_relu2": [_P, _L, _P],
+        "oe_gelu": [_P, _L, _P],
         "oe_tanh_rows": [_P, _P, _L, _P],
         "oe_head_gate": [_P, _P, _L, _P, _L, _P, _I, _I, _I, _I, _I, _I, _F, _P],
         "oe_rot_norm_kv_write": [_P, _L, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P],
@@ -69,6 +71,7 @@ _SIGNATURES = {
         "oe_prev_token_update": [_P, _P, _P, _P, _I, _P],
         "oe_pass_entry_add": [_P, _P, _P, _L, _I, _P],
         "oe_scale_rows": [_P, _L, _F, _P],
+        "oe_softcap_rows": [_P, _L, _F, _P],
     },
     "general_delta": {
         "oe_gdelta_padded_dk": [_I],
@@ -80,7 +83,8 @@ _SIGNATURES = {
         "oe_retention_chunks": [_P, _P, _P, _L, _I, _I, _I, _P, _P, _I, _F, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P],
     },
     "moe": {
-        "oe_moe_route": [_P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _I, _P, _P],
+        "oe_moe_route": [_P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _I, _P, _I, _I, _P],
+        "oe_moe_dense_relu2": [_P, _P, _I, _I, _I, _I, _P],
         "oe_moe_dense_act": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P],
     },
     "stream": {
@@ -114,7 +118,7 @@ _SIGNATURES = {
     },
 }
 _TYPED = {"oe_embed_gather", "oe_rmsnorm", "oe_rope_kv_write", "oe_swiglu", "oe_gemm_simple", "oe_attn_paged",
-          "oe_relu2", "oe_tanh_rows", "oe_rot_norm_kv_write", "oe_token_shift_mix", "oe_last_rows_to_state",
+          "oe_relu2", "oe_gelu", "oe_layernorm", "oe_moe_dense_relu2", "oe_tanh_rows", "oe_rot_norm_kv_write", "oe_token_shift_mix", "oe_last_rows_to_state",
           "oe_rope_split_kv_write", "oe_attn_split", "oe_moe_dense_act", "oe_group_rmsnorm", "oe_poly_norm",
           "oe_side_gate", "oe_latent_write", "oe_attn_latent", "oe_head_matmul", "oe_dyt_norm", "oe_pair_embed",
           "oe_qkv_norm_rot_write", "oe_unrotate_heads"}
@@ -215,6 +219,18 @@ def rmsnorm(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, eps: float) -> No
            "rmsnorm")
 
 
+def layernorm(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float) -> None:
+    """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b, x float32 [rows, D], w and b float32 [D]."""
+    _dev(y, x, w, b)
+    for t, n in ((x, "x"), (w, "w"), (b, "b")):
+        _f32c(t, n)
+    rows, D = x.shape
+    if y.shape != x.shape or not y.is_contiguous() or w.numel() != D or b.numel() != D:
+        raise KernelError("layernorm: y contiguous of x's shape, w and b one value per column")
+    _check(_fn("elementwise", "oe_layernorm", y.dtype)(_ptr(y), _ptr(x), _ptr(w), _ptr(b), rows, D, float(eps), _stream()),
+           "layernorm")
+
+
 def rope_kv_write(qkv: torch.Tensor, cos: torch.Tensor | None, sin: torch.Tensor | None,
                   cache: torch.Tensor | None, tables: torch.Tensor, tok_seq: torch.Tensor,
                   tok_pos: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, has_kv: bool) -> None:
@@ -291,7 +307,8 @@ def gemm_simple(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, accumulate:
 def attn_paged(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, tables: torch.Tensor,
                tok_seq: torch.Tensor, tok_pos: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
                window: int, scale: float, sink: bool = False) -> None:
-    """out[t] = attention of token t's query heads over keys (pos-window, pos] of its sequence.
+    """out[t] = attention of token t's query heads over keys (pos-window, pos] of its sequence (window 0:
+    all keys up to pos; -n: the keys of the chunk of n positions that pos lies in).
 
     q [T, >= H hd] (row stride free, e.g. a view of the qkv buffer), out [T, H hd].
     sink: the softmax's denominator gets one added (a key of score 0 without a value)."""
@@ -349,6 +366,14 @@ def relu2_(a: torch.Tensor) -> None:
     if not a.is_contiguous() or a.dtype not in _SUFFIX:
         raise KernelError("relu2: a contiguous float32 or bfloat16 tensor expected")
     _check(_fn("rowwise", "oe_relu2", a.dtype)(_ptr(a), a.numel(), _stream()), "relu2")
+
+
+def gelu_(a: torch.Tensor) -> None:
+    """a = a (1 + erf(a / sqrt 2)) / 2 in place."""
+    _dev(a)
+    if not a.is_contiguous() or a.dtype not in _SUFFIX:
+        raise KernelError("gelu: a contiguous float32 or bfloat16 tensor expected")
+    _check(_fn("rowwise", "oe_gelu", a.dtype)(_ptr(a), a.numel(), _stream()), "gelu")
 
 
 def tanh_rows(y: torch.Tensor, x: torch.Tensor) -> None:
@@ -634,6 +659,15 @@ def scale_rows(x: torch.Tensor, s: float) -> None:
     _check(_fn("tokenwise", "oe_scale_rows")(_ptr(x), x.numel(), float(s), _stream()), "scale_rows")
 
 
+def softcap_rows(x: torch.Tensor, cap: float) -> None:
+    """x = cap tanh(x / cap); x float32, contiguous."""
+    _dev(x)
+    _f32c(x, "x")
+    if not cap > 0:
+        raise KernelError("softcap_rows: the cap must be positive")
+    _check(_fn("tokenwise", "oe_softcap_rows")(_ptr(x), x.numel(), float(cap), _stream()), "softcap_rows")
+
+
 # ---------------------------------------------------------------------------------------- general_delta.cu
 
 def gdelta_padded_dk(dk: int) -> int:
@@ -739,15 +773,20 @@ def retention_scratch(n_tokens: int, n_seqs: int, heads: int, dk: int, dv: int) 
 
 # ---------------------------------------------------------------------------------------- moe.cu
 
+_ROUTE_MODES = {"softmax": 0, "sigmoid": 1, "softmax_all": 2}
+
+
 def moe_route(z: torch.Tensor, n_experts: int, top: int, has_gate, dense: torch.Tensor, tok_seq: torch.Tensor,
               idx: torch.Tensor | None = None, wt: torch.Tensor | None = None, weights: str = "softmax",
-              bias: torch.Tensor | None = None) -> None:
+              bias: torch.Tensor | None = None, groups: tuple | None = None) -> None:
     """From router logits z float32 [T, >= E (+ 1)]: dense [T, E (+ 1)] float32 gets each chosen expert's weight
     (zero elsewhere) and, with has_gate, sigmoid of column E in its last column (has_gate "one": the constant 1, a
     shared expert without a gate; z needs no column for it); idx int32 [T, top] and wt float32 [T, top] receive the
     choice itself when given.  weights "softmax": the softmax over the `top` largest logits alone; "sigmoid": each
     chosen expert's own sigmoid(logit), not renormalised.  bias (float32 [E], with "sigmoid" only): the choice is by
-    sigmoid(logit) + bias, the weights stay the sigmoids."""
+    sigmoid(logit) + bias, the weights stay the sigmoids.  weights "softmax_all": the softmax over all experts, the chosen
+    scores divided by their sum (+ 1e-20).  groups (count, keep): the experts stand in `count` equal runs, only experts of
+    the `keep` runs with the best single expert can be chosen."""
     _dev(z, dense, tok_seq, idx, wt, bias)
     if bias is not None:
         _f32c(bias, "bias")
@@ -758,8 +797,11 @@ def moe_route(z: torch.Tensor, n_experts: int, top: int, has_gate, dense: torch.
     T = z.shape[0]
     W = n_experts + int(bool(has_gate))
     gate = 2 if has_gate == "one" else int(bool(has_gate))
-    if weights not in ("softmax", "sigmoid"):
-        raise KernelError(f"moe_route: weights must be softmax or sigmoid, got {weights!r}")
+    if weights not in _ROUTE_MODES:
+        raise KernelError(f"moe_route: weights must be one of {', '.join(_ROUTE_MODES)}, got {weights!r}")
+    n_groups, keep = groups or (0, 0)
+    if groups and (n_groups < 1 or n_experts % n_groups or not 1 <= keep <= n_groups or top > keep * (n_experts // n_groups)):
+        raise KernelError(f"moe_route: {n_experts} experts in {n_groups} groups of which {keep} stay cannot give {top}")
     if z.dtype != torch.float32 or z.stride(1) != 1 or z.shape[1] < (n_experts if gate == 2 else W) \
             or tuple(dense.shape) != (T, W):
         raise KernelError("moe_route: z float32 [T, >= E (+1)] and dense [T, E (+1)] expected")
@@ -772,8 +814,19 @@ def moe_route(z: torch.Tensor, n_experts: int, top: int, has_gate, dense: torch.
     for t in (idx, wt):
         if t is not None and tuple(t.shape) != (T, top):
             raise KernelError("moe_route: idx and wt must be [T, top]")
-    _check(_fn("moe", "oe_moe_route")(_ptr(z), z.stride(0), n_experts, top, gate, int(weights == "sigmoid"), _ptr(idx), _ptr(wt),
-                                      _ptr(dense), _ptr(tok_seq), T, _ptr(bias), _stream()), "moe_route")
+    _check(_fn("moe", "oe_moe_route")(_ptr(z), z.stride(0), n_experts, top, gate, _ROUTE_MODES[weights], _ptr(idx), _ptr(wt),
+                                      _ptr(dense), _ptr(tok_seq), T, _ptr(bias), int(n_groups), int(keep), _stream()), "moe_route")
+
+
+def moe_dense_relu2(u: torch.Tensor, dense: torch.Tensor, ff: int) -> None:
+    """u[t, c] = max(u[t, c], 0)^2 * dense[t, c // ff] in place (experts without a gate, side by side)."""
+    _dev(u, dense)
+    _f32c(dense, "dense")
+    T, F = u.shape
+    if not u.is_contiguous() or u.dtype not in _SUFFIX or ff < 1 or F % ff or dense.shape[0] != T or dense.shape[1] < F // ff:
+        raise KernelError("moe_dense_relu2: u contiguous [T, E ff] and dense [T, >= E] expected")
+    _check(_fn("moe", "oe_moe_dense_relu2", u.dtype)(_ptr(u), _ptr(dense), T, F, ff, dense.shape[1], _stream()),
+           "moe_dense_relu2")
 
 
 def moe_dense_act(a: torch.Tensor, gu: torch.Tensor, dense: torch.Tensor, n_experts: int, ff: int,

@@ -604,7 +604,8 @@ def attention_split(out, q, kcache, vcache, tables, ctx, n_heads: int, n_kv_head
     kcache [pages, G, PAGE, dk], vcache [pages, G, PAGE, dv]; vcache None: the values are the first dv columns of the
     key rows.  sinks (float32 [H] or None): exp(sinks[h]) joins head h's denominator, without key or value.  unrotate
     ((cos, sin) float32 [positions, dv/2] or None): every head's result is turned back by its query's position, pair
-    (m, m + dv/2), before it is stored (by the merge kernel when the keys are split)."""
+    (m, m + dv/2), before it is stored (by the merge kernel when the keys are split).  window -n: the keys of the chunk of
+    n positions that the query lies in."""
     uc, us = ops._unrotate_tables(unrotate, dv, "attention_split")
     if sinks is not None and (sinks.dtype != torch.float32 or not sinks.is_contiguous() or sinks.numel() != n_heads):
         raise ops.KernelError("attention_split: sinks must be float32, one value per query head")
@@ -627,7 +628,7 @@ def attention_split(out, q, kcache, vcache, tables, ctx, n_heads: int, n_kv_head
     # would leave SMs idle; the partial sums go through float32 scratch and a merge kernel.
     n_splits, partial = 1, None
     if ctx.all_decode and ctx.n_tokens == ctx.n_seqs:
-        keys = min(window, ctx.max_kvlen) if window else ctx.max_kvlen
+        keys = min(abs(window), ctx.max_kvlen) if window else ctx.max_kvlen
         n_splits = max(1, min(keys // PAGE + 1, (2 * _sm_count()) // max(1, ctx.n_seqs * n_kv_heads), 32))
         if n_splits > 1:
             partial = torch.empty(ctx.n_seqs * n_heads * n_splits * (dv + 2), dtype=torch.float32, device=out.device)

@@ -4,6 +4,7 @@
 //   rmsnorm_add        dst (+)= coef * (y / sqrt(mean(y^2) + eps)) * w        (all float32), optionally with a
 //                      copy of the new dst rounded to bfloat16 (the next sublayer's input)
 //   relu2              a = max(a, 0)^2 in place
+//   gelu               a = a (1 + erf(a / sqrt 2)) / 2 in place
 //   tanh_rows          y = tanh(x), float32 in, compute type out
 //   head_gate          out[t, h, :] = [o / sqrt(mean(o^2) + eps)] * [w] * act(gate)   per head
 //   rot_norm_kv_write  q, k rotated on pairs (2i, 2i+1) of their first `dims` dimensions, then divided
@@ -88,6 +89,14 @@ __global__ void relu2_kernel(T* a, size_t total) {
         const float v = fmaxf(to_f32(a[i]), 0.f);
         a[i] = from_f32<T>(v * v);
     }
+}
+
+template <typename T>
+__global__ void gelu_kernel(T* a, size_t total) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
+        a[i] = from_f32<T>(oe_gelu(to_f32(a[i])));
 }
 
 template <typename T>
@@ -278,6 +287,15 @@ int oe_relu2_f32(float* a, long long total, cudaStream_t st) {
 int oe_relu2_bf16(bf16* a, long long total, cudaStream_t st) {
     if (total <= 0) return 0;
     return oe_launch(relu2_kernel<bf16>, dim3(flat_blocks((size_t)total)), dim3(256), 0, st, a, (size_t)total);
+}
+
+int oe_gelu_f32(float* a, long long total, cudaStream_t st) {
+    if (total <= 0) return 0;
+    return oe_launch(gelu_kernel<float>, dim3(flat_blocks((size_t)total)), dim3(256), 0, st, a, (size_t)total);
+}
+int oe_gelu_bf16(bf16* a, long long total, cudaStream_t st) {
+    if (total <= 0) return 0;
+    return oe_launch(gelu_kernel<bf16>, dim3(flat_blocks((size_t)total)), dim3(256), 0, st, a, (size_t)total);
 }
 
 int oe_tanh_rows_f32(float* y, const float* x, long long total, cudaStream_t st) {

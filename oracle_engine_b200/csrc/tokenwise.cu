@@ -10,6 +10,7 @@
 //   pass_entry_add      x += e + s  (e [rows, D] float32 or null, s [D] float32): what a looped group of layers adds
 //                       to the stream before a pass
 //   scale_rows          x *= s, float32 in place (a constant on the logits)
+//   softcap_rows        x = cap tanh(x / cap), float32 in place (a cap on the logits)
 #include "common.cuh"
 
 namespace {
@@ -116,6 +117,14 @@ __global__ void __launch_bounds__(256) scale_rows_kernel(float* x, size_t total,
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) x[i] *= s;
 }
 
+__global__ void __launch_bounds__(256) softcap_rows_kernel(float* x, size_t total, float cap) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const float inv = 1.f / cap;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
+        x[i] = cap * tanhf(x[i] * inv);
+}
+
 inline unsigned blocks_for(size_t items) {
     size_t blocks = (items + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
@@ -172,6 +181,11 @@ int oe_pass_entry_add(float* x, const float* e, const float* s, long long rows, 
 int oe_scale_rows(float* x, long long total, float s, cudaStream_t st) {
     if (total <= 0) return 0;
     return oe_launch(scale_rows_kernel, dim3(blocks_for((size_t)total)), dim3(256), 0, st, x, (size_t)total, s);
+}
+int oe_softcap_rows(float* x, long long total, float cap, cudaStream_t st) {
+    if (total <= 0) return 0;
+    if (!(cap > 0.f)) return OE_ERR_UNSUPPORTED;
+    return oe_launch(softcap_rows_kernel, dim3(blocks_for((size_t)total)), dim3(256), 0, st, x, (size_t)total, cap);
 }
 
 }  // extern "C"

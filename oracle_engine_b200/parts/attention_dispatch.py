@@ -1,5 +1,6 @@
 """Which attention kernels a step uses: chosen by precision, head size and whether the
-step is a prompt or single decoded tokens; never by the data.
+step is a prompt or single decoded tokens; never by the data.  `window` is a span as the kernels
+take it: 0 every key, n > 0 the last n, -n the query's own chunk of n (parts/spec.py: mask_span).
 
 float32, and head sizes the tensor-core kernels do not take, use the one-path kernel of
 csrc/attention.cu; bfloat16 uses the tensor-core prefill kernel and the split-KV decode
@@ -49,10 +50,12 @@ def attend(rt, out, qkv, cache, ctx, H, KVH, hd, window, scale, sink: bool = Fal
     ops.attn_paged(out, qkv, cache.kv, cache.tables, ctx.tok_seq, ctx.tok_pos, H, KVH, hd, window, scale, sink)
 
 
-def split_mixer_core(rt, out, qkv, cos, sin, rot, kcache, vcache, tables, ctx, H, G, dk, dv, window, scale, cap) -> None:
+def split_mixer_core(rt, out, qkv, cos, sin, rot, kcache, vcache, tables, ctx, H, G, dk, dv, window, scale, cap,
+                     has_kv: bool = True) -> None:
     """Rotation, cache write and attention of an attention mixer whose keys and values have head sizes of their
-    own and lie in two cache tensors, with a cap on the scores (parts/capped_attention.py)."""
-    ops.rope_split_kv_write(qkv, cos, sin, rot, kcache, vcache, tables, ctx.tok_seq, ctx.tok_pos, H, G, dk, dv, True)
+    own and lie in two cache tensors, with a cap on the scores (parts/capped_attention.py).  has_kv False: qkv holds
+    queries only and the cache is another entry's."""
+    ops.rope_split_kv_write(qkv, cos, sin, rot, kcache, vcache, tables, ctx.tok_seq, ctx.tok_pos, H, G, dk, dv, has_kv)
     split_attend(rt, out, qkv, kcache, vcache, tables, ctx, H, G, dk, dv, window, scale, cap)
 
 

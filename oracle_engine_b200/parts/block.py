@@ -5,6 +5,7 @@ outputs into the float32 residual stream themselves (fused into their last produ
 their OUTPUT is normed before it is added; a sublayer adds its output into a zeroed float32 buffer.
 `pre_norm_scaled`: x += m * s1 * mixer(norm(x)); x += m * s2 * ffn(norm(x)) with m one constant and s1, s2 one
 weight per channel each (a layer scale).
+`parallel_sublayers`: h = norm(x); x += mixer(h) + ffn(h): one norm, both sublayers read its output.
 `sandwich`: x += norm_1b(mixer(norm_1(x))); x += norm_2b(ffn(norm_2(x))): a norm before and after every sublayer;
 optionally followed by a per-token side input (`TokenSide`) and an average over the depth (`DepthAverage`)."""
 from __future__ import annotations
@@ -45,6 +46,35 @@ class PreNormBlock:
             self.feed_forward.forward(h, x, ctx)
         if rt is not None:
             rt.next_weights = None
+
+
+@BLOCKS.register("parallel_sublayers")
+class ParallelSublayersBlock:
+    """h = norm(x); x <- x + (mixer(h) + ffn(h)) (the feed-forward is optional).  Both sublayers add into the stream; h
+    was taken before either did."""
+
+    def __init__(self, mixer, feed_forward, mixer_norm, ffn_norm=None):
+        if mixer_norm is None or ffn_norm is not None:
+            raise ValueError("parallel_sublayers: one norm for both sublayers")
+        self.mixer, self.feed_forward, self.norm = mixer, feed_forward, mixer_norm
+
+    def parts(self):
+        return [p for p in (self.norm, self.mixer, self.feed_forward) if p is not None]
+
+    def first_weights(self):
+        return _first_weights(self.mixer)
+
+    def forward(self, x, ctx, cache, state, owns_cache=True):
+        rt = self.mixer.rt
+        after = rt.next_weights
+        h = self.norm.forward(x)
+        if self.feed_forward is not None:
+            rt.next_weights = _first_weights(self.feed_forward)
+        self.mixer.forward(h, x, ctx, cache, state, owns_cache)
+        if self.feed_forward is not None:
+            rt.next_weights = after
+            self.feed_forward.forward(h, x, ctx)
+        rt.next_weights = None
 
 
 @BLOCKS.register("norm_after")

@@ -2,7 +2,8 @@
 
 `token_embedding`: x = E[token] as float32 (core/model.cpp:352-358); an id outside the
 table is an error, not clamped.  `lm_head`: logits = W x in float32, W a separate matrix
-or, when tied, the embedding table (core/model.cpp:482-492); an optional constant `scale` multiplies the logits.
+or, when tied, the embedding table (core/model.cpp:482-492); an optional constant `scale` multiplies the logits,
+an optional `softcap` c bounds them, c tanh(z / c).
 `pair_hash_embedding`: x = E[token] * scale + P[hash(previous token, token)], a second table indexed by a hash of
 the token and the one before it; the previous token is per-sequence state."""
 from __future__ import annotations
@@ -92,7 +93,8 @@ class PairHashEmbedding(Part):
 
 @HEADS.register("lm_head")
 class LMHead(Part):
-    """params: vocab_size, hidden_size, tied, name, scale (a constant the logits are multiplied by; default 1);
+    """params: vocab_size, hidden_size, tied, name, scale (a constant the logits are multiplied by; default 1),
+    softcap (c: the logits become c tanh(z / c); 0 or None: no cap);
     `embedding` is handed in when tied."""
     graph_safe = True
 
@@ -104,6 +106,7 @@ class LMHead(Part):
         self.name = prefix + self.params.get("name", "lm_head.weight")
         self.embedding = self.params.get("embedding")
         self.scale = float(self.params.get("scale", 1.0) or 1.0)
+        self.softcap = float(self.params.get("softcap") or 0.0)
         self.weight = None
 
     def tensors(self):
@@ -123,4 +126,6 @@ class LMHead(Part):
         matmul_nt(self.rt, logits, xn, self.weight)
         if self.scale != 1.0:
             ops.scale_rows(logits, self.scale)
+        if self.softcap > 0:
+            ops.softcap_rows(logits, self.softcap)
         return logits

@@ -1,7 +1,8 @@
 """Feed-forward `swiglu`: g = Wg h, u = Wu h, a = g/(1+exp(-g)) * u, x += Wd a  (dense, no
 routing).  Reference: core/model.cpp:452-473 and :636-643.  The gate and up projections
 are fused into one matrix product at load ([Wg; Wu]).
-Feed-forward `relu2`: a = max(Wu h, 0)^2, x += Wd a (dense, no gate)."""
+Feed-forwards `relu2` and `gelu`: a = max(Wu h, 0)^2 or a = g(Wu h) with the exact gelu
+g(z) = z (1 + erf(z / sqrt 2)) / 2, x += Wd a (dense, no gate)."""
 from __future__ import annotations
 
 import torch
@@ -100,8 +101,19 @@ class SquaredReLU(Part):
         """overwrite: the output is written into `residual` (float32) instead of added."""
         a = self.rt.buffer("relu2.a", h.shape[0], self.FF)
         matmul_nt(self.rt, a, h, self.w_up)
-        ops.relu2_(a)
+        self._activate(a)
         matmul_nt(self.rt, residual, a, self.w_down, accumulate=not overwrite)
+
+    def _activate(self, a):
+        ops.relu2_(a)
+
+
+@FEED_FORWARDS.register("gelu")
+class GeluMLP(SquaredReLU):
+    """params: hidden_size, intermediate_size, tensor_names (optional overrides of "up" and "down")."""
+
+    def _activate(self, a):
+        ops.gelu_(a)
 
 
 @FEED_FORWARDS.register("poly_norm_mlp")

@@ -78,7 +78,8 @@ class DecoderModel:
 
     # ------------------------------------------------------------------ cache / state needs
     def cache_needs(self):
-        """Per schedule entry: the CacheNeed of its mixer, or None if it owns no cache."""
+        """Per schedule entry: the CacheNeed of its mixer, or None if it owns no cache.  An entry that other entries
+        read from keeps what any of them still sees: readers may have masks of their own."""
         out = []
         for e in self.schedule:
             need = self.layers[e.layer].mixer.cache_need()
@@ -86,9 +87,10 @@ class DecoderModel:
         for i, e in enumerate(self.schedule):
             if e.cache_from is not None:
                 mine = self.layers[e.layer].mixer.cache_need()
-                if mine != out[e.cache_from]:
+                if mine is None or mine.tensors != out[e.cache_from].tensors:
                     raise ValueError(f"schedule[{i}] reads the cache of entry {e.cache_from}, whose layout "
                                      f"{out[e.cache_from]} differs from its own {mine}")
+                out[e.cache_from] = out[e.cache_from].joined(mine)
         return out
 
     def state_needs(self):

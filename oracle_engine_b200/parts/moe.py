@@ -9,6 +9,12 @@ scales those: silu(w_e g) * (w_e u)); the shared expert may be added without a g
 sigmoid(z_e) + a learned bias per expert while the weights stay the sigmoids; the experts' unit may be clamped and
 shifted, g = min(Wgate h, L), u = clamp(Wup h, -L, L), E_e(h) = Wdown_e (g * sigmoid(1.702 g) * (u + 1)).
 
+Choice by groups (`groups`, a variant of both kinds): the experts stand in `count` equal runs, a run's score is its best
+expert's, and only experts of the `keep` best runs can be chosen.
+
+Feed-forward `moe_relu2`: experts without a gate, E_e(h) = Wdown_e max(Wup_e h, 0)^2; by default the weights are the
+softmax over ALL experts, the chosen ones divided by their sum (+ 1e-20).
+
 How it is computed: the experts stand side by side.  One product with all gate and up matrices (the shared expert's
 behind the routed ones), one kernel that applies silu(gate) * up and multiplies each expert's columns by the token's
 weight for that expert (zero where it was not chosen, sigmoid(Wsg h) for the shared one), and one product with all
@@ -28,6 +34,18 @@ from .registry import FEED_FORWARDS, Part
 from .spec import TensorDecl
 
 
+def _groups(raw, experts: int, top: int):
+    """(count, keep) of a choice by groups, or None."""
+    if not raw:
+        return None
+    n, keep = int(raw["count"]), int(raw["keep"])
+    if n < 1 or experts % n or not 1 <= keep <= n:
+        raise ValueError(f"a mixture of experts: {experts} experts do not stand in {n} equal groups of which {keep} stay")
+    if top > keep * (experts // n):
+        raise ValueError(f"a mixture of experts: {keep} groups of {experts // n} experts cannot give {top}")
+    return n, keep
+
+
 @FEED_FORWARDS.register("moe_swiglu")
 class MoESwiGLU(Part):
     graph_safe = True
@@ -37,7 +55,7 @@ class MoESwiGLU(Part):
     sigmoid(logit), not renormalised), weight_on ("output", the default: y = sum w_e E_e(h); "input": y = sum E_e(w_e h)),
     shared_gate (default True: the shared expert's output times sigmoid(Wsg h); False: added as it is), choice_bias
     (True: a tensor of one value per expert is added to the sigmoids for the choice alone; needs router_weights
-    "sigmoid"), activation ("silu", the default, or "clamped" with `limit`), tensor_names (optional overrides of
+    "sigmoid"), activation ("silu", the default, or "clamped" with `limit`), groups (None, or {"count", "keep"}), tensor_names (optional overrides of
     "expert" (a format with {e}), "router", "shared", "shared_gate", "choice_bias")."""
 
     def __init__(self, params, prefix, runtime):
@@ -50,8 +68,9 @@ class MoESwiGLU(Part):
         self.router_weights = self.params.get("router_weights") or "softmax"
         self.weight_on = self.params.get("weight_on") or "output"
         self.shared_gate = bool(self.params.get("shared_gate", True)) and self.sff > 0
-        if self.router_weights not in ("softmax", "sigmoid") or self.weight_on not in ("output", "input"):
-            raise ValueError("moe_swiglu: router_weights is softmax or sigmoid, weight_on is output or input")
+        self.groups = _groups(self.params.get("groups"), self.E, self.top)
+        if self.router_weights not in ("softmax", "sigmoid", "softmax_all") or self.weight_on not in ("output", "input"):
+            raise ValueError("moe_swiglu: router_weights is softmax, sigmoid or softmax_all, weight_on is output or input")
         self.choice_bias = bool(self.params.get("choice_bias", False))
         self.activation = self.params.get("activation") or "silu"
         self.limit = float(self.params.get("limit") or 0.0)
@@ -118,10 +137,69 @@ class MoESwiGLU(Part):
         matmul_nt(self.rt, z, h, self.w_route)                  # float32 sums and output on both paths
         dense = self.rt.buffer("moe.dense", T, self.E + (1 if self.sff else 0), dtype=torch.float32)
         ops.moe_route(z, self.E, self.top, (True if self.shared_gate else "one") if self.sff else False, dense,
-                      ctx.tok_seq, weights=self.router_weights, bias=self.bias)
+                      ctx.tok_seq, weights=self.router_weights, bias=self.bias, groups=self.groups)
         gu = self.rt.buffer("moe.gu", T, 2 * self.F)
         matmul_nt(self.rt, gu, h, self.w_gu)
         a = self.rt.buffer("moe.a", T, self.F)
         ops.moe_dense_act(a, gu, dense, self.E, self.ff, scale_input=self.weight_on == "input", act=self.activation,
                           limit=self.limit)
+        matmul_nt(self.rt, residual, a, self.w_down, accumulate=not overwrite)
+
+
+@FEED_FORWARDS.register("moe_relu2")
+class MoEReLU2(Part):
+    graph_safe = True
+    can_overwrite = True
+    """params: hidden_size, num_experts, top, expert_size, groups (None, or {"count", "keep"}), router_weights
+    ("softmax_all", the default, "softmax" or "sigmoid", as csrc/ops.py: moe_route), tensor_names (optional overrides of
+    "expert" (a format with {e}) and "router")."""
+
+    def __init__(self, params, prefix, runtime):
+        super().__init__(params, prefix, runtime)
+        self.D = int(self._need("hidden_size"))
+        self.E = int(self._need("num_experts"))
+        self.top = int(self._need("top"))
+        self.ff = int(self._need("expert_size"))
+        self.groups = _groups(self.params.get("groups"), self.E, self.top)
+        self.router_weights = self.params.get("router_weights") or "softmax_all"
+        if not 1 <= self.top <= self.E <= 1024:
+            raise ValueError(f"moe_relu2: top {self.top} of {self.E} experts (up to 1,024 are supported)")
+        names = {"expert": "mlp.e{e}.", "router": "mlp.router", **self.params.get("tensor_names", {})}
+        self.names = {k: prefix + v for k, v in names.items()}
+        self.F = self.E * self.ff
+        self.w_route = self.w_up = self.w_down = None
+
+    def tensors(self):
+        out = []
+        for e in range(self.E):
+            p = self.names["expert"].format(e=e)
+            out += [TensorDecl(p + "up", (self.ff, self.D)), TensorDecl(p + "down", (self.D, self.ff))]
+        return out + [TensorDecl(self.names["router"], (self.E, self.D))]
+
+    def load(self, get):
+        to = self.rt.to_compute
+        ex = [self.names["expert"].format(e=e) for e in range(self.E)]
+        self.w_up = torch.cat([to(get(p + "up")) for p in ex], 0).contiguous()
+        self.w_down = torch.cat([to(get(p + "down")) for p in ex], 1).contiguous()
+        self.w_route = to(get(self.names["router"]))
+
+    def weight_bytes(self):
+        return sum(t.numel() * t.element_size() for t in (self.w_up, self.w_down, self.w_route) if t is not None)
+
+    def flops(self, start, count):
+        return count * 2.0 * self.D * (2 * self.F + self.E)
+
+    def first_weights(self):
+        return self.w_route
+
+    def forward(self, h, residual, ctx, overwrite: bool = False):
+        """overwrite: the output is written into `residual` (float32) instead of added."""
+        T = h.shape[0]
+        z = self.rt.buffer("moe.z", T, self.E, dtype=torch.float32)
+        matmul_nt(self.rt, z, h, self.w_route)                  # float32 sums and output on both paths
+        dense = self.rt.buffer("moe.dense", T, self.E, dtype=torch.float32)
+        ops.moe_route(z, self.E, self.top, False, dense, ctx.tok_seq, weights=self.router_weights, groups=self.groups)
+        a = self.rt.buffer("moe.a", T, self.F)
+        matmul_nt(self.rt, a, h, self.w_up)
+        ops.moe_dense_relu2(a, dense, self.ff)
         matmul_nt(self.rt, residual, a, self.w_down, accumulate=not overwrite)

@@ -5,7 +5,8 @@ sublayer's float32 OUTPUT and added, times coef, into another float32 tensor (la
 a sublayer returns instead of what it reads).  With `groups` > 1 the row is cut into that many equal consecutive parts
 and each part is divided by its own root mean square (the weight still spans the whole row).
 `dynamic_tanh`: y = tanh(alpha x) * w + b with one scalar alpha and the vectors w, b: a norm that computes no
-mean and no variance, so every value of a row is normed by itself."""
+mean and no variance, so every value of a row is normed by itself.
+`layer_norm`: y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b."""
 from __future__ import annotations
 
 from ..csrc import ops
@@ -62,6 +63,35 @@ class RMSNorm(Part):
             ops.group_rmsnorm_add(dst, y, self.weight, self.eps, self.groups, coef, accumulate, cast)
         else:
             ops.rmsnorm_add(dst, y, self.weight, self.eps, coef, accumulate, cast)
+
+
+@NORMS.register("layer_norm")
+class LayerNorm(Part):
+    graph_safe = True
+    """params: size, eps, name (the weight's tensor name under the prefix), bias (tensor name; default: the weight's
+    name + ".b")."""
+
+    def __init__(self, params, prefix, runtime):
+        super().__init__(params, prefix, runtime)
+        self.size = int(self._need("size"))
+        self.eps = float(self._need("eps"))
+        base = self._need("name")
+        self.name, self.bias_name = prefix + base, prefix + (self.params.get("bias") or base + ".b")
+        self.weight = self.bias = None
+
+    def tensors(self):
+        return [TensorDecl(self.name, (self.size,), "ones_normal"), TensorDecl(self.bias_name, (self.size,))]
+
+    def load(self, get):
+        self.weight, self.bias = self.rt.to_f32(get(self.name)), self.rt.to_f32(get(self.bias_name))
+
+    def weight_bytes(self):
+        return 0 if self.weight is None else 2 * self.weight.numel() * self.weight.element_size()
+
+    def forward(self, x):
+        y = self.rt.empty(*x.shape)
+        ops.layernorm(y, x, self.weight, self.bias, self.eps)
+        return y
 
 
 @NORMS.register("dynamic_tanh")

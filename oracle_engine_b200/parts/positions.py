@@ -44,25 +44,42 @@ def rotary_inv_freq(head_dim: int, theta: float, scaling: dict | None) -> torch.
 
 @POSITIONS.register("rotary")
 class Rotary(Part):
-    """params: head_dim, theta, scaling (None or the llama3 dict), max_positions."""
+    """params: head_dim, theta, scaling (None or the llama3 dict), max_positions, dims (how many dimensions of a head are
+    turned, at frequencies theta^(-2i/dims); default head_dim).  With dims < head_dim the tables still have head_dim / 2
+    columns, the ones behind dims / 2 at angle zero (`head_order` says which dimensions a mixer puts there)."""
 
     def __init__(self, params, prefix, runtime):
         super().__init__(params, prefix, runtime)
         self.head_dim = int(self._need("head_dim"))
         if self.head_dim % 2:
             raise ValueError(f"rotary: head_dim {self.head_dim} must be even")
+        self.dims = int(self.params.get("dims", self.head_dim))
+        if self.dims % 2 or not 0 <= self.dims <= self.head_dim:
+            raise ValueError(f"rotary: {self.dims} turned dimensions must be even and at most head_dim {self.head_dim}")
         self.max_positions = int(self._need("max_positions"))
-        self.inv_freq = rotary_inv_freq(self.head_dim, float(self._need("theta")), self.params.get("scaling"))
+        self.inv_freq = rotary_inv_freq(self.dims, float(self._need("theta")), self.params.get("scaling"))
         self.cos = self.sin = None
 
     def tables(self):
         """(cos, sin), float32 [max_positions, head_dim/2] on the device."""
         if self.cos is None:
             pos = torch.arange(self.max_positions, dtype=torch.float64)
-            ang = pos[:, None] * self.inv_freq[None, :]
+            freq = torch.cat([self.inv_freq, torch.zeros((self.head_dim - self.dims) // 2, dtype=torch.float64)])
+            ang = pos[:, None] * freq[None, :]
             self.cos = torch.cos(ang).to(torch.float32).to(self.rt.device).contiguous()
             self.sin = torch.sin(ang).to(torch.float32).to(self.rt.device).contiguous()
         return self.cos, self.sin
+
+    def head_order(self) -> list | None:
+        """None, or, when only the first `dims` dimensions of a head are turned (i paired with i + dims/2), the order
+        that puts every turned pair at (j, j + head_dim/2) and the untouched dimensions, in pairs of angle zero, behind
+        them: kernels that rotate whole heads by halves then rotate exactly the first `dims`.  A score is a sum over
+        the dimensions, so a query and a key that are both kept in this order score as before."""
+        if self.dims == self.head_dim:
+            return None
+        r, half = self.dims // 2, self.head_dim // 2
+        rest = list(range(self.dims, self.head_dim))
+        return list(range(r)) + rest[:half - r] + list(range(r, self.dims)) + rest[half - r:]
 
 
 @POSITIONS.register("rotary_pairs")

@@ -67,11 +67,34 @@ class CacheNeed:
     and a page of one outer index is one block).  Attention keeps one tensor "kv" of shape
     (2, kv_heads, head_dim); a mixer that keeps one latent vector per token would declare
     (("latent", (rank,)),), keys and values of different widths two tensors.
-    `kind`: "full" (every position) or "window" (the last `window` of them; older pages are
-    given back).  Entries with equal needs share one group of storage and page tables."""
+    `kind`: "full" (every position), "window" (the last `window` of them; older pages are
+    given back) or "chunk" (those of the query's own chunk of `window` positions, counted from
+    position 0; the pages of finished chunks are given back).  `also`: (kind, window) pairs of
+    further readers of the same rows: what any of them still sees is kept.
+    Entries with equal needs share one group of storage and page tables."""
     kind: str
     tensors: tuple
     window: int = 0
+    also: tuple = ()
+
+    def first_position(self, pos: int) -> int:
+        """The oldest position that a query at `pos`, or at any later one, still reads."""
+        first = pos
+        for kind, n in ((self.kind, self.window),) + self.also:
+            if kind == "full":
+                return 0
+            first = min(first, max(0, pos - n + 1) if kind == "window" else pos - pos % n)
+        return first
+
+    def joined(self, other: "CacheNeed") -> "CacheNeed":
+        """The need of rows that both this need's owner and the mixer of `other` read."""
+        mine, theirs = ((self.kind, self.window),) + self.also, ((other.kind, other.window),) + other.also
+        if set(theirs) <= set(mine):
+            return self
+        if any(kind == "full" for kind, _ in mine + theirs):
+            return CacheNeed("full", self.tensors)
+        rest = sorted(set(mine + theirs) - {(self.kind, self.window)})
+        return CacheNeed(self.kind, self.tensors, self.window, tuple(rest))
 
     def elements_per_token(self) -> int:
         n = 0
@@ -83,9 +106,37 @@ class CacheNeed:
         return n
 
 
-def attention_cache_need(kv_heads: int, head_dim: int, window: int = 0) -> CacheNeed:
+def span_need(tensors: tuple, span: int) -> CacheNeed:
+    """The need of an attention whose mask is `span` as the kernels take it (csrc/common.cuh: oe_first_key): 0 every
+    key, n > 0 the last n keys, -n the keys of the query's own chunk of n."""
+    return CacheNeed("window" if span > 0 else "chunk" if span < 0 else "full", tensors, abs(int(span)))
+
+
+def attention_cache_need(kv_heads: int, head_dim: int, span: int = 0) -> CacheNeed:
     """Keys and values of grouped-query attention: one tensor "kv", per page [2, kv_heads, PAGE, head_dim]."""
-    return CacheNeed("window" if window else "full", (("kv", (2, int(kv_heads), int(head_dim))),), int(window))
+    return span_need((("kv", (2, int(kv_heads), int(head_dim))),), span)
+
+
+def mask_span(window, chunk) -> int:
+    """An attention's `window` and `chunk` parameters (0 or None: no such mask) as one span."""
+    window, chunk = int(window or 0), int(chunk or 0)
+    if window < 0 or chunk < 0 or (window and chunk):
+        raise ValueError(f"an attention has a window or chunks of a positive size, not both: {window}, {chunk}")
+    return window if window else -chunk
+
+
+def visible_keys(span: int, context: int) -> int:
+    """How many keys the newest of `context` tokens sees."""
+    return min(context, span) if span > 0 else (context - 1) % -span + 1 if span < 0 else context
+
+
+def visible_pairs(span: int, start: int, count: int) -> float:
+    """The (query, key) pairs of `count` tokens at positions start .. start + count - 1."""
+    tri = lambda n: n * (n + 1) / 2.0                                    # noqa: E731
+    upto = lambda n: tri(n) if not span else \
+        tri(min(n, span)) + span * max(0, n - span) if span > 0 else \
+        (n // -span) * tri(-span) + tri(n % -span)                       # noqa: E731
+    return upto(start + count) - upto(start)
 
 
 @dataclass(frozen=True)
