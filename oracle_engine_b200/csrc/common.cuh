@@ -129,6 +129,56 @@ __device__ __forceinline__ float warp_max(float v) {
 // z times the normal distribution function: the exact gelu.
 __device__ __forceinline__ float oe_gelu(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
+// What a product does to its float32 sums before it stores them as bfloat16: the features (weight rows) from `from` on
+// go through `act` and are then multiplied by a per-token weight of their group of `ff` features, w[token * ld +
+// (feature - from) / ff] (w null: by nothing); the features before `from` are stored as they are.
+struct OeEpilogue {
+    int act;                   // 0 none, 1 exact gelu, 2 squared ReLU
+    int from, ff;
+    long long ld;
+    const float* w;            // written by an earlier kernel of the stream: read only behind pdl_wait()
+};
+__device__ __forceinline__ float oe_activate(int act, float v) {
+    if (act == 1) return oe_gelu(v);
+    const float r = fmaxf(v, 0.f);
+    return r * r;
+}
+// N consecutive features of one token, feature0 .. feature0 + N - 1; those from n_features on are not stored.
+template <int N>
+__device__ __forceinline__ void oe_epilogue_row(const OeEpilogue& e, float (&v)[N], int token, int feature0, int n_features) {
+    if (feature0 + N <= e.from) return;
+    if (e.w == nullptr) {
+#pragma unroll
+        for (int j = 0; j < N; j++)
+            if (feature0 + j >= e.from) v[j] = oe_activate(e.act, v[j]);
+        return;
+    }
+    const float* row = e.w + (long long)token * e.ld;
+    int group = max(feature0 - e.from, 0) / e.ff;
+    float weight = feature0 < n_features ? row[group] : 0.f;
+#pragma unroll
+    for (int j = 0; j < N; j++) {
+        const int f = feature0 + j - e.from;
+        if (f < 0) continue;
+        if (f >= (group + 1) * e.ff) {
+            group++;
+            weight = feature0 + j < n_features ? row[group] : 0.f;
+        }
+        v[j] = oe_activate(e.act, v[j]) * weight;
+    }
+}
+__device__ __forceinline__ float oe_epilogue_one(const OeEpilogue& e, float v, int token, int feature) {
+    if (feature < e.from) return v;
+    v = oe_activate(e.act, v);
+    return e.w == nullptr ? v : v * e.w[(long long)token * e.ld + (feature - e.from) / e.ff];
+}
+// The host side of the four arguments: false if they make no sense.
+static inline bool oe_epilogue_ok(const OeEpilogue& e, int out_kind, int n_features) {
+    if (e.act == 0) return e.w == nullptr;
+    return (e.act == 1 || e.act == 2) && out_kind == 0 && e.from >= 0 && e.from <= n_features &&
+           (e.w == nullptr || (e.ff > 0 && e.ld >= (n_features - e.from + e.ff - 1) / e.ff));
+}
+
 // Sum over a block in a fixed order (warp shuffles, then warp 0 over the warp totals);
 // every thread gets the result.  `red` holds 32 floats of shared memory.
 __device__ __forceinline__ float block_sum(float v, float* red) {

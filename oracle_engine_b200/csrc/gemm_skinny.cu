@@ -40,7 +40,7 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
 template <int NT, int WARPS, int UNROLL>
 __global__ void __launch_bounds__(WARPS * 32)
 gemm_skinny_kernel(void* C, const bf16* A, const bf16* __restrict__ W,
-                   int M, int N, int K, long long lda, long long ldc, int out_kind, int late_trigger) {
+                   int M, int N, int K, long long lda, long long ldc, int out_kind, int late_trigger, const OeEpilogue epi) {
     __shared__ float red[WARPS][ROWS][8 * NT + 1];
     __shared__ float total[ROWS][8 * NT + 1];
     if (!late_trigger) pdl_launch_dependents();
@@ -118,7 +118,7 @@ gemm_skinny_kernel(void* C, const bf16* A, const bf16* __restrict__ W,
         const int row = row0 + r;
         if (tok >= M || row >= N) continue;
         const float v = total[r][tok];
-        if (out_kind == 0) ((bf16*)C)[(size_t)tok * ldc + row] = __float2bfloat16_rn(v);
+        if (out_kind == 0) ((bf16*)C)[(size_t)tok * ldc + row] = __float2bfloat16_rn(epi.act ? oe_epilogue_one(epi, v, tok, row) : v);
         else if (out_kind == 1) ((float*)C)[(size_t)tok * ldc + row] = v;
         else if (out_kind == 2) ((float*)C)[(size_t)tok * ldc + row] += v;
         else if (!(r & 1)) {
@@ -140,11 +140,14 @@ int oe_gemm_skinny_supported(const void* A, const void* W, int M, int N, int K, 
 }
 
 // out_kind: 0 bf16, 1 float32, 2 float32 accumulate, 3 bf16 silu(gate)*up on interleaved rows (C is [M, N/2]).
-// early: bit 0 start early, bit 1 trigger late (see below).
+// early: bit 0 start early, bit 1 trigger late (see below).  act ..: what happens to the sums (common.cuh: OeEpilogue).
 int oe_gemm_skinny_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int K, long long lda, long long ldc,
-                        int out_kind, int early, cudaStream_t st) {
+                        int out_kind, int early, int act, int act_from, const float* act_w, int act_ff, long long act_ld,
+                        cudaStream_t st) {
     if (!oe_gemm_skinny_supported(A, W, M, N, K, lda)) return OE_ERR_UNSUPPORTED;
     if (out_kind < 0 || out_kind > 3 || (out_kind == 3 && (N & 1))) return OE_ERR_UNSUPPORTED;
+    const OeEpilogue epi = {act, act_from, act_ff, act_ld, act_w};
+    if (!oe_epilogue_ok(epi, out_kind, N)) return OE_ERR_UNSUPPORTED;
     const int blocks = (N + ROWS - 1) / ROWS;
     // early bit 0: the kernel may start (and request its first weights) while the kernel before it
     // drains.  early bit 1: this kernel releases the kernel after it only when its CTAs have
@@ -161,7 +164,7 @@ int oe_gemm_skinny_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int
     // with more loads in flight.
 #define OE_SKINNY_LAUNCH(NT, WARPS, UNROLL)                                                                        \
     return oe_launch_ex((early & 1) != 0, gemm_skinny_kernel<NT, WARPS, UNROLL>, dim3(blocks), dim3(WARPS * 32), 0, st, C, A, \
-                        W, M, N, K, lda, ldc, out_kind, (early >> 1) & 1)
+                        W, M, N, K, lda, ldc, out_kind, (early >> 1) & 1, epi)
     if (M > 8) {
         // 9 to 16 tokens, chosen inside the 28-layer decode step (16 sequences: 2.11 ms with 8 warps x 3 loads
         // for every shape, 1.96 ms with these)

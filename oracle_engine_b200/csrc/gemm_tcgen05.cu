@@ -172,6 +172,7 @@ struct GemmArgs {
     int stages;
     int swap;                   // 1: C[b_row, a_row] (A = weights); 0: C[a_row, b_row] (A = activations)
     int out_kind;               // 0 bf16 store, 1 float32 store, 2 float32 accumulate, 3 bf16 silu(gate)*up
+    OeEpilogue epi;             // what happens to the sums before a bf16 store (out_kind 0)
     int splits;
     int tiles_a, tiles_b;       // output tiles along the A and the B operand
     int streamk;                // 1: the CTAs share the k-blocks of the first sk_tiles tiles equally (see ItemIter)
@@ -208,8 +209,17 @@ __device__ __forceinline__ float silu_mul(float gate, float up) { return (gate /
 // out_kind 3: rows of the weight matrix alternate gate, up (g0, u0, g1, u1, ...); the output
 // is silu(gate) * up as bf16, half as many features.
 template <int NC>
-__device__ __forceinline__ void emit(const GemmArgs& g, int a_row, int b_row0, const float (&v)[NC]) {
+__device__ __forceinline__ void emit(const GemmArgs& g, int a_row, int b_row0, float (&v)[NC]) {
     const bool a_ok = a_row < g.rows_a;
+    if (g.epi.act && a_ok) {
+        if (g.swap) {
+#pragma unroll
+            for (int j = 0; j < NC; j++)
+                if (b_row0 + j < g.rows_b) v[j] = oe_epilogue_one(g.epi, v[j], b_row0 + j, a_row);
+        } else {
+            oe_epilogue_row<NC>(g.epi, v, a_row, b_row0, g.rows_b);
+        }
+    }
     if (g.swap) {
         if (g.out_kind == 3) {
 #pragma unroll
@@ -627,7 +637,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
                     for (int q = 0; q < 2; q++)
                         if ((q == 0 || two) && tile_b * g.n_tile + c0 + 16 * q < g.rows_b)
-                            emit<16>(g, a_row, tile_b * g.n_tile + c0 + 16 * q, reinterpret_cast<const float(&)[16]>(acc[16 * q]));
+                            emit<16>(g, a_row, tile_b * g.n_tile + c0 + 16 * q, reinterpret_cast<float(&)[16]>(acc[16 * q]));
                 }
                 asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
                 __syncwarp();
@@ -865,16 +875,20 @@ int oe_gemm_tc_counters() { return 4096; }
 
 // C[M,N] (+)= A[M,K] . W[N,K]^T ; out_kind: 0 bf16, 1 float32, 2 float32 accumulate,
 // 3: W's rows alternate gate/up and C[M,N/2] = silu(gate) * up as bf16 (ldc counts C's elements).
+// act ..: what happens to the sums before a bf16 store (common.cuh: OeEpilogue).
 // workspace: float32 scratch of ws_bytes bytes, counters: n_counters zeroed ints (both may be null: no split).
 int oe_gemm_tc_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int K, long long lda, long long ldc,
                     int out_kind, float* workspace, long long ws_bytes, int* counters, int n_counters,
-                    int sm_count, cudaStream_t st) {
+                    int sm_count, int act, int act_from, const float* act_w, int act_ff, long long act_ld,
+                    cudaStream_t st) {
     if (!oe_gemm_tc_supported(A, W, M, N, K, lda)) return OE_ERR_UNSUPPORTED;
     if (out_kind < 0 || out_kind > 3 || (out_kind == 3 && (N & 1))) return OE_ERR_UNSUPPORTED;
     int rc = get_encode();
     if (rc) return rc;
     GemmArgs g;
     g.C = C; g.ldc = ldc; g.K = K; g.out_kind = out_kind;
+    g.epi = OeEpilogue{act, act_from, act_ff, act_ld, act_w};
+    if (!oe_epilogue_ok(g.epi, out_kind, N)) return OE_ERR_UNSUPPORTED;
     g.workspace = workspace; g.counters = counters; g.splits = 1; g.streamk = 0; g.sk_tiles = 0; g.cluster = 1;
     g.atoms = 1;
     g.wait_ns = g_wait_ns; g.withhold_release = g_withhold_release;

@@ -55,6 +55,7 @@ struct PairArgs {
     int acc_cols;                  // tensor-memory columns between the two accumulators (n_tile rounded up to 32)
     int stages;
     int out_kind;                  // 0 bf16 store, 1 float32 store, 2 float32 accumulate, 3 bf16 silu(gate)*up
+    OeEpilogue epi;                // what happens to the sums before a bf16 store (out_kind 0)
     int tiles_m, tiles_n;          // tiles of 256 rows and of n_tile columns
 };
 
@@ -169,8 +170,9 @@ __device__ __forceinline__ void red_add4(float* p, float a, float b, float c, fl
 }
 
 // 16 consecutive columns (col0 ..) of output row `row`.  out_kind 3: the columns alternate gate, up.
-__device__ __forceinline__ void emit16(const PairArgs& g, int row, int col0, const float (&v)[16]) {
+__device__ __forceinline__ void emit16(const PairArgs& g, int row, int col0, float (&v)[16]) {
     if (row >= g.M) return;
+    if (g.epi.act) oe_epilogue_row<16>(g.epi, v, row, col0, g.N);
     const bool full = col0 + 16 <= g.N;
     if (g.out_kind == 3) {
         const long long base = (long long)row * g.ldc + (col0 >> 1);
@@ -408,9 +410,11 @@ int oe_gemm_pair_supported(const void* A, const void* W, int M, int N, int K, lo
 
 // C[M,N] (+)= A[M,K] . W[N,K]^T ; out_kind: 0 bf16, 1 float32, 2 float32 accumulate,
 // 3: W's rows alternate gate/up and C[M,N/2] = silu(gate) * up as bf16 (ldc counts C's elements).
+// act ..: what happens to the sums before a bf16 store (common.cuh: OeEpilogue).
 // max_tile: 0, or an upper limit for the tile's columns (for tests).
 int oe_gemm_pair_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int K, long long lda, long long ldc,
-                      int out_kind, int max_tile, cudaStream_t st) {
+                      int out_kind, int max_tile, int act, int act_from, const float* act_w, int act_ff, long long act_ld,
+                      cudaStream_t st) {
     if (!oe_gemm_pair_supported(A, W, M, N, K, lda)) return OE_ERR_UNSUPPORTED;
     if (out_kind < 0 || out_kind > 3 || (out_kind == 3 && (N & 1))) return OE_ERR_UNSUPPORTED;
     int rc = get_encode();
@@ -433,6 +437,8 @@ int oe_gemm_pair_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int K
     }
     PairArgs g;
     g.C = C; g.ldc = ldc; g.M = M; g.N = N; g.K = K; g.out_kind = out_kind;
+    g.epi = OeEpilogue{act, act_from, act_ff, act_ld, act_w};
+    if (!oe_epilogue_ok(g.epi, out_kind, N)) return OE_ERR_UNSUPPORTED;
     g.tiles_m = (M + 2 * BLOCK_M - 1) / (2 * BLOCK_M);
     // The tile width (a multiple of 16) with the shortest rounds of clusters at the measured time of a
     // pair's k-block: 230, 249, 284, 310 and 365 ns from 128, 160, 192, 224 and 256 columns on, and a

@@ -72,6 +72,10 @@ def knobs(**kw):
             _lib().oe_gemm_tc_waits(c_longlong(int(KNOBS.gemm_waits[0])), int(KNOBS.gemm_waits[1]))
 
 
+_EPILOGUE = [c_int, c_int, c_void_p, c_int, c_longlong]      # act, act_from, weights, features per group, row stride
+ACTIVATIONS = {None: 0, "gelu": 1, "relu2": 2}
+
+
 def _lib():
     lib = _state.get("gemm")
     if lib is None:
@@ -79,7 +83,7 @@ def _lib():
         lib.oe_gemm_tc_supported.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_longlong]
         lib.oe_gemm_tc_supported.restype = c_int
         lib.oe_gemm_tc_bf16.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong,
-                                        c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p]
+                                        c_int, c_void_p, c_longlong, c_void_p, c_int, c_int] + _EPILOGUE + [c_void_p]
         lib.oe_gemm_tc_bf16.restype = c_int
         lib.oe_gemm_tc_prefetch.argtypes = [c_void_p, c_longlong]
         lib.oe_gemm_tc_prefetch.restype = None
@@ -154,7 +158,7 @@ def _pair():
     if lib is None:
         lib = _build.load("gemm_pair")
         lib.oe_gemm_pair_bf16.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong,
-                                          c_int, c_int, c_void_p]
+                                          c_int, c_int] + _EPILOGUE + [c_void_p]
         lib.oe_gemm_pair_bf16.restype = c_int
         lib.oe_gemm_pair_error.restype = c_int
         _state["pair"] = lib
@@ -166,7 +170,7 @@ def _skinny():
     if lib is None:
         lib = _build.load("gemm_skinny")
         lib.oe_gemm_skinny_bf16.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong,
-                                            c_int, c_int, c_void_p]
+                                            c_int, c_int] + _EPILOGUE + [c_void_p]
         lib.oe_gemm_skinny_bf16.restype = c_int
         _state["skinny"] = lib
     return lib
@@ -176,11 +180,15 @@ NEXT_WEIGHTS_L2_BYTES = 8 << 20     # see gemm(then=)
 
 
 def gemm(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, accumulate: bool = False, split_k: bool = True,
-         swiglu: bool = False, kernel: str = "auto", early: int = 0, then: torch.Tensor | None = None) -> None:
+         swiglu: bool = False, kernel: str = "auto", early: int = 0, then: torch.Tensor | None = None,
+         act: str | None = None, act_from: int = 0, group_weights: tuple | None = None) -> None:
     """out (+)= a @ w.T, a [M, K] and w [N, K] bfloat16; out bfloat16 or float32 [M, N].
 
     swiglu: w's rows alternate gate and up rows (g0, u0, g1, u1, ...) and out [M, N/2]
     bfloat16 receives silu(gate) * up, computed in float32 in the epilogue.
+    act ("gelu" or "relu2", out bfloat16): the columns of out from act_from on are act(sum), computed in the epilogue from
+    the float32 sums; group_weights (w float32 [M, >= groups], ff): column c of them is then multiplied by
+    w[row, (c - act_from) // ff].
     kernel: "auto" (weight-streaming kernel for a handful of rows, see uses_skinny, the two-SM tcgen05
     kernel from PAIR_MIN_TOKENS rows, the one-SM tcgen05 kernel otherwise),
     "tcgen05", "pair" or "skinny".
@@ -210,14 +218,27 @@ def gemm(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, accumulate: bool =
         kind = 1
     else:
         raise KernelError("gemm: output must be bfloat16 or float32")
+    epilogue = [ACTIVATIONS[act], 0, None, 0, 0]
+    if act is not None:
+        if kind != 0 or not 0 <= act_from <= N:
+            raise KernelError("gemm: an activation needs a bfloat16 output and starts at one of its columns")
+        epilogue[1] = int(act_from)
+        if group_weights is not None:
+            gw, ff = group_weights
+            if gw.dtype != torch.float32 or gw.stride(1) != 1 or gw.shape[0] < M or ff < 1 or \
+                    gw.shape[1] * ff < N - act_from or gw.device != a.device:
+                raise KernelError("gemm: group weights must be float32 [M, groups], one column per ff features")
+            epilogue[2:] = [gw.data_ptr(), int(ff), gw.stride(0)]
+    elif group_weights is not None:
+        raise KernelError("gemm: group weights come with an activation")
     if kernel == "skinny" or (kernel == "auto" and uses_skinny(M, N, K, kind)):
         code = _skinny().oe_gemm_skinny_bf16(out.data_ptr(), a.data_ptr(), w.data_ptr(), M, N, K, a.stride(0),
-                                             out.stride(0), kind, int(early), ops._stream())
+                                             out.stride(0), kind, int(early), *epilogue, ops._stream())
         ops._check(code, "gemm_skinny", (M, N, K))
         return
     if kernel == "pair" or (kernel == "auto" and uses_pair(M, N, K, KNOBS.sm_count or None)):
         code = _pair().oe_gemm_pair_bf16(out.data_ptr(), a.data_ptr(), w.data_ptr(), M, N, K, a.stride(0), out.stride(0),
-                                         kind, int(KNOBS.pair_max_tile), ops._stream())
+                                         kind, int(KNOBS.pair_max_tile), *epilogue, ops._stream())
         ops._check(code, "gemm_pair", (M, N, K))
         return
     ws, counters, sms = _scratch(a.device)
@@ -227,7 +248,7 @@ def gemm(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, accumulate: bool =
     code = _lib().oe_gemm_tc_bf16(out.data_ptr(), a.data_ptr(), w.data_ptr(), M, N, K, a.stride(0), out.stride(0), kind,
                                   ws.data_ptr() if split_k else None, ws.numel() * 4,
                                   counters.data_ptr() if split_k else None, counters.numel(), sms,
-                                  ops._stream())
+                                  *epilogue, ops._stream())
     ops._check(code, "gemm_tc", (M, N, K))
 
 

@@ -87,15 +87,21 @@ class GQAAttention(Part):
     def first_weights(self):
         return self.w_qkv
 
-    def forward(self, h, residual, ctx, cache, state, owns_cache=True):
+    joint_weight = "w_qkv"         # parts/block.py: JoinedInput
+
+    def forward(self, h, residual, ctx, cache, state, owns_cache=True, projected=None):
+        """projected: Wqkv h (Wq h first), computed by the caller; the rotation works in it."""
         if self.reads_cache and owns_cache:
             raise ValueError("gqa_attention: a layer without key and value projections must read another entry's cache")
         T = h.shape[0]
         q_width = self.H * self.hd
         width = q_width + (2 * self.KVH * self.hd if owns_cache else 0)
-        qkv = self.rt.empty(T, width)
-        # how the products are chained to their neighbours in the stream: parts/linear.py
-        matmul_nt(self.rt, qkv, h, self.w_qkv[:width], early=chain_flags("mixer_in", T))
+        if projected is not None:
+            qkv = projected[:, :width]
+        else:
+            qkv = self.rt.empty(T, width)
+            # how the products are chained to their neighbours in the stream: parts/linear.py
+            matmul_nt(self.rt, qkv, h, self.w_qkv[:width], early=chain_flags("mixer_in", T))
         cos, sin = self.position.tables() if self.position is not None else (None, None)
         from . import attention_dispatch as ad
         o = self.rt.empty(T, q_width)

@@ -48,26 +48,75 @@ class PreNormBlock:
             rt.next_weights = None
 
 
+class JoinedInput(Part):
+    """One product for what two sublayers read from the same input: [Wmixer; Wffn] h, the feed-forward's columns
+    activated (and weighted, for experts) in the product's epilogue.  It takes the place of two products wherever the
+    tensor-core kernels serve the shapes and both sublayers offer it: a part with `joint_weight` (the attribute that
+    holds its first matrix) whose `forward` takes `projected`; the feed-forward also has `joint_epilogue(h, ctx)`, which
+    runs what must come first (a router) and returns (activation, group weights or None).  It has no tensors of its
+    own: once both sublayers have loaded theirs, the two matrices move into one and stay views of it."""
+    graph_safe = True
+
+    def __init__(self, mixer, feed_forward):
+        super().__init__({}, "", mixer.rt)
+        self.sublayers = (mixer, feed_forward)
+        self.weight = None
+        self.split = 0
+
+    def load(self, get):
+        mixer, ffn = self.sublayers
+        self.weight = None
+        if ffn is None or not (hasattr(mixer, "joint_weight") and hasattr(ffn, "joint_epilogue")):
+            return
+        a, b = getattr(mixer, mixer.joint_weight), getattr(ffn, ffn.joint_weight)
+        # rows of 16-byte pieces: the operands of the products that read the two parts start on such a boundary
+        if self.rt.dtype != torch.bfloat16 or not self.rt.tensor_cores or a.shape[1] % 8 or a.shape[0] % 8 or b.shape[0] % 8:
+            return
+        self.split = a.shape[0]
+        self.weight = torch.cat([a, b], 0)
+        setattr(mixer, mixer.joint_weight, self.weight[:self.split])
+        setattr(ffn, ffn.joint_weight, self.weight[self.split:])
+
+    def forward(self, h, ctx):
+        """(what the mixer takes as `projected`, what the feed-forward takes)."""
+        from ..csrc import ops_tc
+        from .linear import chain_flags
+        T = h.shape[0]
+        act, weights = self.sublayers[1].joint_epilogue(h, ctx)
+        y = self.rt.buffer("joined", T, self.weight.shape[0])
+        ops_tc.gemm(y, h, self.weight, act=act, act_from=self.split, group_weights=weights, early=chain_flags("mixer_in", T))
+        return y[:, :self.split], y[:, self.split:]
+
+
 @BLOCKS.register("parallel_sublayers")
 class ParallelSublayersBlock:
     """h = norm(x); x <- x + (mixer(h) + ffn(h)) (the feed-forward is optional).  Both sublayers add into the stream; h
-    was taken before either did."""
+    was taken before either did.  On the tensor-core path the first products of the two are one (`JoinedInput`)."""
 
     def __init__(self, mixer, feed_forward, mixer_norm, ffn_norm=None):
         if mixer_norm is None or ffn_norm is not None:
             raise ValueError("parallel_sublayers: one norm for both sublayers")
         self.mixer, self.feed_forward, self.norm = mixer, feed_forward, mixer_norm
+        self.joined = JoinedInput(mixer, feed_forward)
 
     def parts(self):
-        return [p for p in (self.norm, self.mixer, self.feed_forward) if p is not None]
+        return [p for p in (self.norm, self.mixer, self.feed_forward, self.joined) if p is not None]
 
     def first_weights(self):
-        return _first_weights(self.mixer)
+        return self.joined.weight if self.joined.weight is not None else _first_weights(self.mixer)
 
     def forward(self, x, ctx, cache, state, owns_cache=True):
         rt = self.mixer.rt
         after = rt.next_weights
         h = self.norm.forward(x)
+        if self.joined.weight is not None:
+            rt.next_weights = None
+            for_mixer, for_ffn = self.joined.forward(h, ctx)
+            self.mixer.forward(h, x, ctx, cache, state, owns_cache, projected=for_mixer)
+            rt.next_weights = after
+            self.feed_forward.forward(h, x, ctx, projected=for_ffn)
+            rt.next_weights = None
+            return
         if self.feed_forward is not None:
             rt.next_weights = _first_weights(self.feed_forward)
         self.mixer.forward(h, x, ctx, cache, state, owns_cache)

@@ -80,15 +80,20 @@ class CappedAttention(Part):
     def first_weights(self):
         return self.w_qkv
 
-    def forward(self, h, residual, ctx, cache, state, owns_cache=True, overwrite: bool = False):
-        """overwrite: the output is written into `residual` (float32) instead of added."""
+    joint_weight = "w_qkv"         # parts/block.py: JoinedInput
+
+    def forward(self, h, residual, ctx, cache, state, owns_cache=True, overwrite: bool = False, projected=None):
+        """overwrite: the output is written into `residual` (float32) instead of added.  projected: Wqkv h (Wq h first),
+        computed by the caller; the rotation works in it."""
         if owns_cache == self.reads_cache:
             raise ValueError("capped_attention: a layer without key and value projections must read another entry's "
                              "cache (and one with them must own its cache)")
         T = h.shape[0]
         qw = self.H * self.dk
-        qkv = self.rt.buffer("capped.qkv", T, self.w_qkv.shape[0])
-        matmul_nt(self.rt, qkv, h, self.w_qkv)
+        qkv = projected
+        if qkv is None:
+            qkv = self.rt.buffer("capped.qkv", T, self.w_qkv.shape[0])
+            matmul_nt(self.rt, qkv, h, self.w_qkv)
         cos, sin = self.position.tables() if self.rot else (None, None)
         kc, vc = cache.tensors["k"], cache.tensors["v"]
         o = self.rt.buffer("capped.o", T, self.H * self.dv)

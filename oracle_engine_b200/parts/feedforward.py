@@ -8,7 +8,7 @@ from __future__ import annotations
 import torch
 
 from ..csrc import ops
-from .linear import chain_flags, matmul_nt
+from .linear import chain_flags, matmul_act, matmul_nt
 from .registry import FEED_FORWARDS, Part
 from .spec import TensorDecl
 
@@ -96,24 +96,30 @@ class SquaredReLU(Part):
         return self.w_up
 
     can_overwrite = True
+    act = "relu2"
 
-    def forward(self, h, residual, ctx, overwrite: bool = False):
-        """overwrite: the output is written into `residual` (float32) instead of added."""
-        a = self.rt.buffer("relu2.a", h.shape[0], self.FF)
-        matmul_nt(self.rt, a, h, self.w_up)
-        self._activate(a)
-        matmul_nt(self.rt, residual, a, self.w_down, accumulate=not overwrite)
+    # what an arrangement that makes one product of both sublayers' inputs asks for (parts/block.py: JoinedInput)
+    joint_weight = "w_up"
 
-    def _activate(self, a):
-        ops.relu2_(a)
+    def joint_epilogue(self, h, ctx):
+        return self.act, None
+
+    def forward(self, h, residual, ctx, overwrite: bool = False, projected=None):
+        """overwrite: the output is written into `residual` (float32) instead of added.  projected: act(Wu h), computed
+        by the caller."""
+        T, a = h.shape[0], projected
+        if a is None:
+            a = self.rt.buffer("updown.a", T, self.FF)
+            matmul_act(self.rt, a, h, self.w_up, self.act, early=chain_flags("ffn_in", T))
+        matmul_nt(self.rt, residual, a, self.w_down, accumulate=not overwrite, early=chain_flags("ffn_out", T),
+                  then=self.rt.next_weights)
 
 
 @FEED_FORWARDS.register("gelu")
 class GeluMLP(SquaredReLU):
     """params: hidden_size, intermediate_size, tensor_names (optional overrides of "up" and "down")."""
 
-    def _activate(self, a):
-        ops.gelu_(a)
+    act = "gelu"
 
 
 @FEED_FORWARDS.register("poly_norm_mlp")

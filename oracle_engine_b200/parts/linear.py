@@ -47,3 +47,22 @@ def matmul_nt(rt, out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, accumulat
             ops_tc.gemm(out, a, w, accumulate=accumulate, early=int(early), then=then)
             return
     ops.gemm_simple(out, a, w, accumulate=accumulate)
+
+
+def matmul_act(rt, out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, act: str, group_weights: tuple | None = None,
+               early: int = 0) -> None:
+    """out = act(a @ w.T), act "gelu" or "relu2", out of the compute dtype; with group_weights (float32 [T, groups], ff;
+    "relu2" only) column c times weights[:, c // ff].  Where a tensor-core product takes the shapes the activation is its
+    epilogue, on the float32 sums; else it is a kernel of its own."""
+    if rt.dtype == torch.bfloat16 and rt.tensor_cores:
+        from ..csrc import ops_tc
+        if ops_tc.gemm_supported(a, w, out):
+            ops_tc.gemm(out, a, w, act=act, group_weights=group_weights, early=int(early))
+            return
+    ops.gemm_simple(out, a, w)
+    if group_weights is not None:
+        if act != "relu2":
+            raise ValueError("group weights go with squared-ReLU experts")
+        ops.moe_dense_relu2(out, *group_weights)
+    else:
+        {"gelu": ops.gelu_, "relu2": ops.relu2_}[act](out)

@@ -29,7 +29,7 @@ from __future__ import annotations
 import torch
 
 from ..csrc import ops
-from .linear import matmul_nt
+from .linear import chain_flags, matmul_act, matmul_nt
 from .registry import FEED_FORWARDS, Part
 from .spec import TensorDecl
 
@@ -192,14 +192,25 @@ class MoEReLU2(Part):
     def first_weights(self):
         return self.w_route
 
-    def forward(self, h, residual, ctx, overwrite: bool = False):
-        """overwrite: the output is written into `residual` (float32) instead of added."""
+    joint_weight = "w_up"
+
+    def joint_epilogue(self, h, ctx):
+        """The routing, and what the up product does with its sums: squared ReLU times the token's weight for the
+        column's expert (zero where it was not chosen)."""
         T = h.shape[0]
         z = self.rt.buffer("moe.z", T, self.E, dtype=torch.float32)
         matmul_nt(self.rt, z, h, self.w_route)                  # float32 sums and output on both paths
         dense = self.rt.buffer("moe.dense", T, self.E, dtype=torch.float32)
         ops.moe_route(z, self.E, self.top, False, dense, ctx.tok_seq, weights=self.router_weights, groups=self.groups)
-        a = self.rt.buffer("moe.a", T, self.F)
-        matmul_nt(self.rt, a, h, self.w_up)
-        ops.moe_dense_relu2(a, dense, self.ff)
-        matmul_nt(self.rt, residual, a, self.w_down, accumulate=not overwrite)
+        return "relu2", (dense, self.ff)
+
+    def forward(self, h, residual, ctx, overwrite: bool = False, projected=None):
+        """overwrite: the output is written into `residual` (float32) instead of added.  projected: the weighted,
+        activated up product, computed by the caller."""
+        T, a = h.shape[0], projected
+        if a is None:
+            act, weights = self.joint_epilogue(h, ctx)
+            a = self.rt.buffer("moe.a", T, self.F)
+            matmul_act(self.rt, a, h, self.w_up, act, weights, early=chain_flags("ffn_in", T))
+        matmul_nt(self.rt, residual, a, self.w_down, accumulate=not overwrite, early=chain_flags("ffn_out", T),
+                  then=self.rt.next_weights)
