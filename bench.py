@@ -6,7 +6,7 @@
     python bench.py --shape 8b --workload baseline      # 32 prompts of 128..4,096 tokens, 256 steps
     python bench.py --profile [--batch 64]              # device time per kind of kernel, on standard error
     python bench.py --impl reference --steps K          # the reference's own benchmark program (CPU)
-    python bench.py --design fuvipel|fovirax|pusunex|bogupel [--beside llama,fovirax] [--widths 1024,2048,3072] [--profile]
+    python bench.py --design fuvipel|fovirax|pusunex|bogupel|goridra [--beside llama,fovirax] [--widths 1024,2048,3072] [--profile]
                                                         # that design beside a Llama of equal width and depth
 
 Prints ONE JSON line.  `value` is decoded tokens per second at the given batch (default
@@ -440,6 +440,21 @@ def bogupel_shape(width: int, layers: int, vocab: int) -> dict:
             "layers": [delta if i % 3 == 2 else att for i in range(layers)]}
 
 
+def goridra_shape(width: int, layers: int, vocab: int) -> dict:
+    """A Goridra of real layer sizes: attention in chunks of 1,024 with heads of 128 (four query heads to a key head, half
+    of each head turned); every second layer reads the keys and values of the one before it; dense feed-forwards of 4 x
+    width on the layers with keys of their own, on the others a mixture of 8 experts of 2/3 x width in four groups of
+    which two stay, two experts chosen; capped logits, the embedding table as the head."""
+    heads = width // 128
+    ff = (2 * width // 3 + 63) // 64 * 64
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+           "mask": {"size": 1024}, "rot": {"dims": 64, "base": 500000.0}}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Goridra", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": [{"type": "attention", "mixer": dict(att, kv_from=i - 1), "mlp": moe} if i % 2 else
+                       {"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": 4 * width}} for i in range(layers)]}
+
+
 def llama_shape(width: int, layers: int, vocab: int) -> dict:
     """The Llama decoder of the same width, depth and vocabulary: heads of 128, four query heads to a key head,
     a SwiGLU of 8/3 x width (the same weights as a two-matrix feed-forward of 4 x width)."""
@@ -458,12 +473,14 @@ def design_compare(args) -> int:
     from oracle_engine_b200.config.bogupel import BogupelConfig
     from oracle_engine_b200.config.fovirax import FoviraxConfig
     from oracle_engine_b200.config.fuvipel import FuvipelConfig
+    from oracle_engine_b200.config.goridra import GoridraConfig
     from oracle_engine_b200.config.pusunex import PusunexConfig
     from oracle_engine_b200.engine.engine import Engine
     designs = {"fuvipel": lambda *a: FuvipelConfig.from_dict(fuvipel_shape(*a)),
                "fovirax": lambda *a: FoviraxConfig.from_dict(fovirax_shape(*a)),
                "pusunex": lambda *a: PusunexConfig.from_dict(pusunex_shape(*a)),
                "bogupel": lambda *a: BogupelConfig.from_dict(bogupel_shape(*a)),
+               "goridra": lambda *a: GoridraConfig.from_dict(goridra_shape(*a)),
                "llama": lambda *a: LlamaConfig.from_dict(llama_shape(*a))}
     beside = [b for b in (args.beside or "llama").split(",") if b and b != args.design]
     unknown = [b for b in beside if b not in designs]
@@ -627,7 +644,7 @@ def main():
     ap.add_argument("--profile", action="store_true",
                     help="print device time per kind of kernel of a prompt step and a decode step on standard error, "
                          "and nothing else")
-    ap.add_argument("--design", default=None, choices=["fuvipel", "fovirax", "pusunex", "bogupel"],
+    ap.add_argument("--design", default=None, choices=["fuvipel", "fovirax", "pusunex", "bogupel", "goridra"],
                     help="measure this design beside the Llama decoder at equal sizes instead of the headline workload")
     ap.add_argument("--beside", default=None, help="the designs to measure beside --design, comma-separated (default llama)")
     ap.add_argument("--widths", default="1024,2048,3072", help="model widths of --design")

@@ -138,39 +138,72 @@ struct OeEpilogue {
     long long ld;
     const float* w;            // written by an earlier kernel of the stream: read only behind pdl_wait()
 };
-__device__ __forceinline__ float oe_activate(int act, float v) {
-    if (act == 1) return oe_gelu(v);
-    const float r = fmaxf(v, 0.f);
-    return r * r;
+// The exact gelu for a result that is rounded to bfloat16, without branches, so that the values of a row overlap:
+// 1 - erf(x) by formula 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical Functions (absolute error 1.5e-7).
+__device__ __forceinline__ float oe_gelu_bf16(float z) {
+    const float x = fabsf(z) * 0.70710678118654752f;
+    const float t = __fdividef(1.f, fmaf(0.3275911f, x, 1.f));
+    float p = fmaf(1.061405429f, t, -1.453152027f);
+    p = fmaf(p, t, 1.421413741f);
+    p = fmaf(p, t, -0.284496736f);
+    p = fmaf(p, t, 0.254829592f);
+    const float h = 0.5f * z * (p * t * __expf(-x * x));          // z times half of what lies beyond |z|
+    return z >= 0.f ? z - h : h;
 }
+template <int N>
+__device__ __forceinline__ void oe_activate(int act, float (&v)[N]) {
+    if (act == 1) {
+#pragma unroll
+        for (int j = 0; j < N; j++) v[j] = oe_gelu_bf16(v[j]);
+    } else {
+#pragma unroll
+        for (int j = 0; j < N; j++) { const float r = fmaxf(v[j], 0.f); v[j] = r * r; }
+    }
+}
+// A token's weight of the group that holds the features [lo, hi) behind `from`: kept while a thread walks along a row.
+struct OeGroupWeight {
+    int lo = 0, hi = 0;
+    float w = 0.f;
+};
 // N consecutive features of one token, feature0 .. feature0 + N - 1; those from n_features on are not stored.
 template <int N>
-__device__ __forceinline__ void oe_epilogue_row(const OeEpilogue& e, float (&v)[N], int token, int feature0, int n_features) {
+__device__ __forceinline__ void oe_epilogue_row(const OeEpilogue& e, float (&v)[N], int token, int feature0, int n_features,
+                                                OeGroupWeight& kept) {
     if (feature0 + N <= e.from) return;
-    if (e.w == nullptr) {
-#pragma unroll
-        for (int j = 0; j < N; j++)
-            if (feature0 + j >= e.from) v[j] = oe_activate(e.act, v[j]);
+    const int b0 = feature0 - e.from;
+    if (b0 >= 0 && e.w == nullptr) {
+        oe_activate(e.act, v);
         return;
     }
     const float* row = e.w + (long long)token * e.ld;
-    int group = max(feature0 - e.from, 0) / e.ff;
-    float weight = feature0 < n_features ? row[group] : 0.f;
-#pragma unroll
-    for (int j = 0; j < N; j++) {
-        const int f = feature0 + j - e.from;
-        if (f < 0) continue;
-        if (f >= (group + 1) * e.ff) {
-            group++;
-            weight = feature0 + j < n_features ? row[group] : 0.f;
+    if (b0 >= 0 && (b0 < kept.lo || b0 + N > kept.hi) && feature0 < n_features) {
+        const int group = b0 / e.ff;
+        if (b0 + N <= (group + 1) * e.ff) {
+            kept.lo = group * e.ff;
+            kept.hi = kept.lo + e.ff;
+            kept.w = row[group];
         }
-        v[j] = oe_activate(e.act, v[j]) * weight;
     }
+    if (b0 >= 0 && b0 >= kept.lo && b0 + N <= kept.hi) {
+        oe_activate(e.act, v);
+#pragma unroll
+        for (int j = 0; j < N; j++) v[j] *= kept.w;
+        return;
+    }
+    // the features lie on both sides of `from` or of a group's edge
+    float u[N];
+#pragma unroll
+    for (int j = 0; j < N; j++) u[j] = v[j];
+    oe_activate(e.act, u);
+#pragma unroll
+    for (int j = 0; j < N; j++)
+        if (b0 + j >= 0 && feature0 + j < n_features) v[j] = e.w == nullptr ? u[j] : u[j] * row[(b0 + j) / e.ff];
 }
 __device__ __forceinline__ float oe_epilogue_one(const OeEpilogue& e, float v, int token, int feature) {
     if (feature < e.from) return v;
-    v = oe_activate(e.act, v);
-    return e.w == nullptr ? v : v * e.w[(long long)token * e.ld + (feature - e.from) / e.ff];
+    float u[1] = {v};
+    oe_activate(e.act, u);
+    return e.w == nullptr ? u[0] : u[0] * e.w[(long long)token * e.ld + (feature - e.from) / e.ff];
 }
 // The host side of the four arguments: false if they make no sense.
 static inline bool oe_epilogue_ok(const OeEpilogue& e, int out_kind, int n_features) {

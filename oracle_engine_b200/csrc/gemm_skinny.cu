@@ -37,7 +37,8 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
 
 // NT: 8-token tiles, 1 (M <= 8) or 2 (M <= 16); WARPS: warps per CTA (they split K);
 // UNROLL: 64-wide k chunks whose weight loads a warp has in flight at once.
-template <int NT, int WARPS, int UNROLL>
+// ACT: the product has an epilogue (common.cuh: OeEpilogue); a form of its own, so that the others stay as they are.
+template <int NT, int WARPS, int UNROLL, bool ACT>
 __global__ void __launch_bounds__(WARPS * 32)
 gemm_skinny_kernel(void* C, const bf16* A, const bf16* __restrict__ W,
                    int M, int N, int K, long long lda, long long ldc, int out_kind, int late_trigger, const OeEpilogue epi) {
@@ -118,7 +119,7 @@ gemm_skinny_kernel(void* C, const bf16* A, const bf16* __restrict__ W,
         const int row = row0 + r;
         if (tok >= M || row >= N) continue;
         const float v = total[r][tok];
-        if (out_kind == 0) ((bf16*)C)[(size_t)tok * ldc + row] = __float2bfloat16_rn(epi.act ? oe_epilogue_one(epi, v, tok, row) : v);
+        if (out_kind == 0) ((bf16*)C)[(size_t)tok * ldc + row] = __float2bfloat16_rn(ACT ? oe_epilogue_one(epi, v, tok, row) : v);
         else if (out_kind == 1) ((float*)C)[(size_t)tok * ldc + row] = v;
         else if (out_kind == 2) ((float*)C)[(size_t)tok * ldc + row] += v;
         else if (!(r & 1)) {
@@ -163,8 +164,11 @@ int oe_gemm_skinny_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int
     // Warps and loads in flight per shape: matrices with many rows do best with small CTAs, long rows
     // with more loads in flight.
 #define OE_SKINNY_LAUNCH(NT, WARPS, UNROLL)                                                                        \
-    return oe_launch_ex((early & 1) != 0, gemm_skinny_kernel<NT, WARPS, UNROLL>, dim3(blocks), dim3(WARPS * 32), 0, st, C, A, \
-                        W, M, N, K, lda, ldc, out_kind, (early >> 1) & 1, epi)
+    return epi.act                                                                                                 \
+        ? oe_launch_ex((early & 1) != 0, gemm_skinny_kernel<NT, WARPS, UNROLL, true>, dim3(blocks), dim3(WARPS * 32), 0, st, C, \
+                       A, W, M, N, K, lda, ldc, out_kind, (early >> 1) & 1, epi)                                   \
+        : oe_launch_ex((early & 1) != 0, gemm_skinny_kernel<NT, WARPS, UNROLL, false>, dim3(blocks), dim3(WARPS * 32), 0, st, C, \
+                       A, W, M, N, K, lda, ldc, out_kind, (early >> 1) & 1, epi)
     if (M > 8) {
         // 9 to 16 tokens, chosen inside the 28-layer decode step (16 sequences: 2.11 ms with 8 warps x 3 loads
         // for every shape, 1.96 ms with these)

@@ -208,16 +208,16 @@ __device__ __forceinline__ float silu_mul(float gate, float up) { return (gate /
 // 32 lanes of a warp together (out_kind 3 exchanges values between neighbouring lanes).
 // out_kind 3: rows of the weight matrix alternate gate, up (g0, u0, g1, u1, ...); the output
 // is silu(gate) * up as bf16, half as many features.
-template <int NC>
-__device__ __forceinline__ void emit(const GemmArgs& g, int a_row, int b_row0, float (&v)[NC]) {
+template <int NC, bool ACT>
+__device__ __forceinline__ void emit(const GemmArgs& g, int a_row, int b_row0, float (&v)[NC], OeGroupWeight& kept) {
     const bool a_ok = a_row < g.rows_a;
-    if (g.epi.act && a_ok) {
+    if (ACT && a_ok) {
         if (g.swap) {
 #pragma unroll
             for (int j = 0; j < NC; j++)
                 if (b_row0 + j < g.rows_b) v[j] = oe_epilogue_one(g.epi, v[j], b_row0 + j, a_row);
         } else {
-            oe_epilogue_row<NC>(g.epi, v, a_row, b_row0, g.rows_b);
+            oe_epilogue_row<NC>(g.epi, v, a_row, b_row0, g.rows_b, kept);
         }
     }
     if (g.swap) {
@@ -379,6 +379,8 @@ __device__ __forceinline__ size_t part_base(const GemmArgs& g, const ItemIter& t
     return ((size_t)p * g.tiles_a * g.tiles_b + (size_t)it.tile_a * g.tiles_b + it.tile_b) * tile_floats;
 }
 
+// ACT: the product has an epilogue (common.cuh: OeEpilogue); a form of its own, so that the others stay as they are.
+template <bool ACT>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const GemmArgs g) {
     extern __shared__ __align__(1024) uint8_t smem_raw[];
@@ -585,6 +587,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 break;                                      // one work item per CTA in this mode
             }
             const bool shared_tile = item.n_parts > 1;      // several work items add up to this tile
+            OeGroupWeight kept;                             // of this thread's row, along the tile's columns
             const int tile_id = tile_a * tiles_b + tile_b;
             // A piece lies in the workspace as [column / 4][row][4] floats: a thread's four columns
             // are one 16-byte access and a warp's accesses are contiguous.
@@ -637,7 +640,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
                     for (int q = 0; q < 2; q++)
                         if ((q == 0 || two) && tile_b * g.n_tile + c0 + 16 * q < g.rows_b)
-                            emit<16>(g, a_row, tile_b * g.n_tile + c0 + 16 * q, reinterpret_cast<float(&)[16]>(acc[16 * q]));
+                            emit<16, ACT>(g, a_row, tile_b * g.n_tile + c0 + 16 * q, reinterpret_cast<float(&)[16]>(acc[16 * q]), kept);
                 }
                 asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
                 __syncwarp();
@@ -666,7 +669,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                         for (int j = 0; j < 4; j++)
                             part[(size_t)j * BLOCK_M] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
                     } else {
-                        emit<16>(g, a_row, tile_b * g.n_tile + c, v);
+                        emit<16, ACT>(g, a_row, tile_b * g.n_tile + c, v, kept);
                     }
                 }
             }
@@ -722,7 +725,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                                 }
                             }
                         }
-                        emit<16>(g, a_row, tile_b * g.n_tile + c0, acc);
+                        emit<16, ACT>(g, a_row, tile_b * g.n_tile + c0, acc, kept);
                     }
                     if (warp == 2 && lane == 0) g.counters[tile_id] = 0;
                 }
@@ -776,7 +779,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                         }
                     }
                 }
-                emit<16>(g, mine ? cl_tile_a * BLOCK_M + row : 0x3fffffff, cl_tile_b * g.n_tile + grp * 16, acc);
+                OeGroupWeight kept;
+                emit<16, ACT>(g, mine ? cl_tile_a * BLOCK_M + row : 0x3fffffff, cl_tile_b * g.n_tile + grp * 16, acc, kept);
             }
         }
         cluster_sync();                               // nobody leaves while its shared memory is read
@@ -841,7 +845,7 @@ int make_map(CUtensorMap* map, const void* ptr, long long rows, long long K, lon
 int max_clusters(int cs) {
     if (cs < 1 || cs > 8) return 0;
     if (g_max_clusters[cs] >= 0) return g_max_clusters[cs];
-    cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
     if (e != cudaSuccess) return -(int)e;
     cudaLaunchConfig_t probe = {};
     probe.gridDim = dim3((unsigned)cs); probe.blockDim = dim3(THREADS); probe.dynamicSmemBytes = 227 * 1024;
@@ -850,7 +854,7 @@ int max_clusters(int cs) {
     pa[0].val.clusterDim.x = (unsigned)cs; pa[0].val.clusterDim.y = 1; pa[0].val.clusterDim.z = 1;
     probe.attrs = pa; probe.numAttrs = 1;
     int n = 0;
-    e = cudaOccupancyMaxActiveClusters(&n, gemm_tc_kernel, &probe);
+    e = cudaOccupancyMaxActiveClusters(&n, gemm_tc_kernel<false>, &probe);
     if (e != cudaSuccess) { cudaGetLastError(); n = 0; }
     g_max_clusters[cs] = n;
     return n;
@@ -1046,13 +1050,14 @@ int oe_gemm_tc_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int K, 
     const size_t smem = (size_t)stages * stage_bytes + sizeof(SharedCtl) + 1024;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (e != cudaSuccess) return (int)e;
         attr_set = true;
     }
     if (g.cluster > 1)
-        return oe_launch_cluster(gemm_tc_kernel, (unsigned)g.cluster, dim3(grid), dim3(THREADS), smem, st, map_a, map_b, g);
-    const int launch_rc = oe_launch(gemm_tc_kernel, dim3(grid), dim3(THREADS), smem, st, map_a, map_b, g);
+        return oe_launch_cluster(g.epi.act ? gemm_tc_kernel<true> : gemm_tc_kernel<false>, (unsigned)g.cluster, dim3(grid), dim3(THREADS), smem, st, map_a, map_b, g);
+    const int launch_rc = oe_launch(g.epi.act ? gemm_tc_kernel<true> : gemm_tc_kernel<false>, dim3(grid), dim3(THREADS), smem, st, map_a, map_b, g);
     return launch_rc;
 }
 

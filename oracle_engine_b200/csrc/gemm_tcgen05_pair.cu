@@ -170,9 +170,10 @@ __device__ __forceinline__ void red_add4(float* p, float a, float b, float c, fl
 }
 
 // 16 consecutive columns (col0 ..) of output row `row`.  out_kind 3: the columns alternate gate, up.
-__device__ __forceinline__ void emit16(const PairArgs& g, int row, int col0, float (&v)[16]) {
+template <bool ACT>
+__device__ __forceinline__ void emit16(const PairArgs& g, int row, int col0, float (&v)[16], OeGroupWeight& kept) {
     if (row >= g.M) return;
-    if (g.epi.act) oe_epilogue_row<16>(g.epi, v, row, col0, g.N);
+    if (ACT) oe_epilogue_row<16>(g.epi, v, row, col0, g.N, kept);
     const bool full = col0 + 16 <= g.N;
     if (g.out_kind == 3) {
         const long long base = (long long)row * g.ldc + (col0 >> 1);
@@ -221,6 +222,8 @@ __device__ __forceinline__ void emit16(const PairArgs& g, int row, int col0, flo
     }
 }
 
+// ACT: the product has an epilogue (common.cuh: OeEpilogue); a form of its own, so that the others stay as they are.
+template <bool ACT>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const PairArgs g) {
     extern __shared__ __align__(1024) uint8_t smem_raw[];
@@ -330,6 +333,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
             const int tile_n = w / g.tiles_m, tile_m = w % g.tiles_m;
             const int row = tile_m * (2 * BLOCK_M) + (int)rank * BLOCK_M + row_in_cta;
             const int buf = lt & 1;
+            OeGroupWeight kept;                            // of this thread's row, along the tile's columns
             if (!mbar_wait(&ctl->tmem_full[buf], (uint32_t)(lt >> 1) & 1u, ctl, 3)) break;
             if (first) { pdl_wait(); first = false; }     // before the first access to C
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -346,7 +350,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
                     float v[16];
 #pragma unroll
                     for (int j = 0; j < 16; j++) v[j] = __uint_as_float(r[h][j]);
-                    emit16(g, row, tile_n * g.n_tile + c0 + 16 * h, v);
+                    emit16<ACT>(g, row, tile_n * g.n_tile + c0 + 16 * h, v, kept);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -422,7 +426,8 @@ int oe_gemm_pair_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int K
     const size_t smem_max = 227 * 1024;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_max);
+        cudaError_t e = cudaFuncSetAttribute(gemm_pair_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_max);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_pair_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_max);
         if (e != cudaSuccess) return (int)e;
         attr_set = true;
     }
@@ -430,7 +435,7 @@ int oe_gemm_pair_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int K
         cudaLaunchConfig_t probe = {};
         probe.gridDim = dim3(2); probe.blockDim = dim3(THREADS); probe.dynamicSmemBytes = smem_max;
         int n = 0;
-        cudaError_t e = cudaOccupancyMaxActiveClusters(&n, gemm_pair_kernel, &probe);
+        cudaError_t e = cudaOccupancyMaxActiveClusters(&n, gemm_pair_kernel<false>, &probe);
         if (e != cudaSuccess) return (int)e;
         if (n < 1) return OE_ERR_UNSUPPORTED;
         g_clusters = n;
@@ -474,7 +479,7 @@ int oe_gemm_pair_bf16(void* C, const bf16* A, const bf16* W, int M, int N, int K
     g.stages = stages;
     const size_t smem = (size_t)stages * stage_bytes + sizeof(SharedCtl) + 1024;
     const int clusters = (int)(n_work < g_clusters ? n_work : g_clusters);
-    return oe_launch(gemm_pair_kernel, dim3(2 * clusters), dim3(THREADS), smem, st, map_a, map_b, g);
+    return oe_launch(g.epi.act ? gemm_pair_kernel<true> : gemm_pair_kernel<false>, dim3(2 * clusters), dim3(THREADS), smem, st, map_a, map_b, g);
 }
 
 // Reads and clears the device-side error flag (0 = no wait ran out).
