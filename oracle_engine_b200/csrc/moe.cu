@@ -12,6 +12,7 @@
 //                   mode 2: the scores are the softmax over ALL experts, the weights the chosen scores over (their sum
 //                   + 1e-20).  n_groups > 0: the experts stand in n_groups equal runs, a run's score is its best
 //                   expert's, and only experts of the `keep` best runs can be chosen.
+//   moe_router      the router's product with bfloat16 inputs and moe_route in one launch (up to 64 rows of weights).
 //   moe_dense_act   gu [T, 2 F] holds, for F = E ff + shared_ff columns, the gate rows and, F columns further, the
 //                   up rows of all experts (expert e owns columns e ff .. (e + 1) ff - 1, the shared expert the last
 //                   shared_ff).  a[t, c] = silu(gate) * up * dense[t, expert of c]: the experts a token did not
@@ -22,15 +23,11 @@
 
 namespace {
 
-__global__ void __launch_bounds__(128)
-moe_route_kernel(const float* z, long long ldz, int E, int top, int has_gate, int mode, int* idx, float* wt, float* dense,
-                 const int* __restrict__ tok_seq, int n_tokens, const float* __restrict__ bias, int n_groups, int keep) {
-    __shared__ unsigned kept_runs[4][32];
-    pdl_launch_dependents();
-    pdl_wait();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t = blockIdx.x * 4 + warp;
-    if (t >= n_tokens) return;
+// One warp routes token t, whose logits are zr (global or shared memory); `kept` is the warp's own 32 words of shared
+// memory (bit g: run g stays in the race).
+__device__ __forceinline__ void route_token(const float* zr, int t, int lane, int E, int top, int has_gate, int mode, int* idx,
+                                            float* wt, float* dense, const int* __restrict__ tok_seq,
+                                            const float* __restrict__ bias, int n_groups, int keep, unsigned* kept) {
     const int W = E + (has_gate ? 1 : 0);
     float* drow = dense + (size_t)t * W;
     for (int e = lane; e < W; e += 32) drow[e] = 0.f;
@@ -42,10 +39,8 @@ moe_route_kernel(const float* z, long long ldz, int E, int top, int has_gate, in
         return;
     }
     __syncwarp();
-    const float* zr = z + (size_t)t * ldz;
     // what the choice goes by: a logit (its order is the softmax's), or sigmoid + bias
     auto score = [&](int e) { return bias ? 1.f / (1.f + expf(-zr[e])) + bias[e] : zr[e]; };
-    unsigned* kept = kept_runs[warp];        // bit g: run g stays in the race
     const int per_run = n_groups > 0 ? E / n_groups : E;
     if (n_groups > 0) {
         kept[lane] = 0u;
@@ -114,6 +109,85 @@ moe_route_kernel(const float* z, long long ldz, int E, int top, int has_gate, in
         if (taken >> i & 1u) drow[e] *= inv;
     if (wt) for (int j = lane; j < top; j += 32) wt[(size_t)t * top + j] *= inv;
     if (has_gate && lane == 0) drow[E] = has_gate == 2 ? 1.f : 1.f / (1.f + expf(-zr[E]));
+}
+
+__global__ void __launch_bounds__(128)
+moe_route_kernel(const float* z, long long ldz, int E, int top, int has_gate, int mode, int* idx, float* wt, float* dense,
+                 const int* __restrict__ tok_seq, int n_tokens, const float* __restrict__ bias, int n_groups, int keep) {
+    __shared__ unsigned kept_runs[4][32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.x * 4 + warp;
+    if (t >= n_tokens) return;
+    route_token(z + (size_t)t * ldz, t, lane, E, top, has_gate, mode, idx, wt, dense, tok_seq, bias, n_groups, keep, kept_runs[warp]);
+}
+
+// The router's product and the routing in one launch, for bfloat16 inputs and up to ROWS (8, 16, 32 or 64) rows of router
+// weights [R, D] (the experts', and the shared expert's gate behind them).  A block takes TOK tokens; its 8 warps share
+// the columns, 256 a warp and turn, a lane 8 of them (16 bytes) of every token and every row; float32 sums, added over
+// the lanes and then over the warps in their order, so that a token's logits do not depend on its neighbours.
+constexpr int ROUTER_WARPS = 8;
+template <int ROWS, int TOK>
+__global__ void __launch_bounds__(ROUTER_WARPS * 32)
+moe_router_kernel(const bf16* h, long long ldh, const bf16* __restrict__ w, int R, int D, int E, int top, int has_gate,
+                  int mode, float* dense, const int* __restrict__ tok_seq, int n_tokens, const float* __restrict__ bias,
+                  int n_groups, int keep) {
+    __shared__ float part[ROUTER_WARPS][TOK][ROWS];
+    __shared__ float z[TOK][ROWS];
+    __shared__ unsigned kept_runs[TOK][32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.x * TOK;
+    float acc[TOK][ROWS];
+#pragma unroll
+    for (int i = 0; i < TOK; i++)
+#pragma unroll
+        for (int r = 0; r < ROWS; r++) acc[i][r] = 0.f;
+    for (int c = (warp * 32 + lane) * 8; c < D; c += ROUTER_WARPS * 256) {
+        float x[TOK][8];
+#pragma unroll
+        for (int i = 0; i < TOK; i++) {
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (t0 + i < n_tokens) v = *reinterpret_cast<const uint4*>(h + (size_t)(t0 + i) * ldh + c);
+            const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&v);
+#pragma unroll
+            for (int j = 0; j < 4; j++) { const float2 f = __bfloat1622float2(p[j]); x[i][2 * j] = f.x; x[i][2 * j + 1] = f.y; }
+        }
+#pragma unroll
+        for (int r = 0; r < ROWS; r++) {
+            if (r >= R) break;
+            const uint4 v = *reinterpret_cast<const uint4*>(w + (size_t)r * D + c);
+            const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&v);
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const float2 f = __bfloat1622float2(p[j]);
+#pragma unroll
+                for (int i = 0; i < TOK; i++) acc[i][r] = fmaf(x[i][2 * j + 1], f.y, fmaf(x[i][2 * j], f.x, acc[i][r]));
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < ROWS; r++) {
+        if (r >= R) break;
+#pragma unroll
+        for (int i = 0; i < TOK; i++) {
+            const float s = warp_sum(acc[i][r]);
+            if (lane == 0) part[warp][i][r] = s;
+        }
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < TOK * R; e += blockDim.x) {
+        float s = 0.f;
+#pragma unroll
+        for (int q = 0; q < ROUTER_WARPS; q++) s += part[q][e / R][e % R];
+        z[e / R][e % R] = s;
+    }
+    __syncthreads();
+    if (warp < TOK && t0 + warp < n_tokens)
+        route_token(z[warp], t0 + warp, lane, E, top, has_gate, mode, nullptr, nullptr, dense, tok_seq, bias, n_groups, keep,
+                    kept_runs[warp]);
 }
 
 // One thread takes 8 consecutive columns of one token (16 bytes of bfloat16) where an expert's columns come in
@@ -235,6 +309,24 @@ int oe_moe_route(const float* z, long long ldz, int E, int top, int has_gate, in
     if (n_groups < 0 || (n_groups > 0 && (E % n_groups || keep < 1 || keep > n_groups))) return OE_ERR_UNSUPPORTED;
     return oe_launch(moe_route_kernel, dim3((n_tokens + 3) / 4), dim3(128), 0, st, z, ldz, E, top, has_gate, mode, idx, wt, dense,
                      tok_seq, n_tokens, bias, n_groups, keep);
+}
+// h [T, D] bfloat16 (rows of ldh), w [R, D] bfloat16 with R = E rows, one more when has_gate is 1.
+int oe_moe_router(const bf16* h, long long ldh, const bf16* w, int D, int E, int top, int has_gate, int mode, float* dense,
+                  const int* tok_seq, int n_tokens, const float* bias, int n_groups, int keep, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
+    const int R = E + (has_gate == 1 ? 1 : 0);
+    if (E < 1 || R > 64 || top < 1 || mode < 0 || mode > 2 || (bias != nullptr && mode != 1)) return OE_ERR_UNSUPPORTED;
+    if (n_groups < 0 || (n_groups > 0 && (E % n_groups || keep < 1 || keep > n_groups))) return OE_ERR_UNSUPPORTED;
+    if (D % 8 || ldh % 8 || (((uintptr_t)h | (uintptr_t)w) & 15)) return OE_ERR_UNSUPPORTED;
+#define OE_ROUTER(ROWS, TOK)                                                                                              \
+    return oe_launch(moe_router_kernel<ROWS, TOK>, dim3((n_tokens + TOK - 1) / TOK), dim3(ROUTER_WARPS * 32), 0, st, h, ldh, w, \
+                     R, D, E, top, has_gate, mode, dense, tok_seq, n_tokens, bias, n_groups, keep)
+    // few tokens: a block each; many: the weights' loads serve several
+    if (R <= 8) { if (n_tokens <= 296) OE_ROUTER(8, 1); OE_ROUTER(8, 4); }
+    if (R <= 16) { if (n_tokens <= 296) OE_ROUTER(16, 1); OE_ROUTER(16, 4); }
+    if (R <= 32) OE_ROUTER(32, 1);
+    OE_ROUTER(64, 1);
+#undef OE_ROUTER
 }
 int oe_moe_dense_relu2_f32(float* u, const float* dense, int n_tokens, int F, int ff, int W, cudaStream_t st) {
     return launch_relu2<float>(u, dense, n_tokens, F, ff, W, st);

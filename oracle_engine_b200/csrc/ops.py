@@ -84,6 +84,7 @@ _SIGNATURES = {
     },
     "moe": {
         "oe_moe_route": [_P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _I, _P, _I, _I, _P],
+        "oe_moe_router": [_P, _L, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _I, _I, _P],
         "oe_moe_dense_relu2": [_P, _P, _I, _I, _I, _I, _P],
         "oe_moe_dense_act": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P],
     },
@@ -776,6 +777,22 @@ def retention_scratch(n_tokens: int, n_seqs: int, heads: int, dk: int, dv: int) 
 _ROUTE_MODES = {"softmax": 0, "sigmoid": 1, "softmax_all": 2}
 
 
+def _route_arguments(n_experts: int, top: int, has_gate, weights: str, bias, groups) -> tuple:
+    """(gate, number of groups, groups that stay), checked."""
+    if bias is not None:
+        _f32c(bias, "bias")
+        if weights != "sigmoid" or bias.numel() != n_experts:
+            raise KernelError("moe_route: a choice bias needs sigmoid weights and one value per expert")
+    if weights not in _ROUTE_MODES:
+        raise KernelError(f"moe_route: weights must be one of {', '.join(_ROUTE_MODES)}, got {weights!r}")
+    if top > n_experts:
+        raise KernelError("moe_route: more experts chosen than there are")
+    n_groups, keep = groups or (0, 0)
+    if groups and (n_groups < 1 or n_experts % n_groups or not 1 <= keep <= n_groups or top > keep * (n_experts // n_groups)):
+        raise KernelError(f"moe_route: {n_experts} experts in {n_groups} groups of which {keep} stay cannot give {top}")
+    return 2 if has_gate == "one" else int(bool(has_gate)), int(n_groups), int(keep)
+
+
 def moe_route(z: torch.Tensor, n_experts: int, top: int, has_gate, dense: torch.Tensor, tok_seq: torch.Tensor,
               idx: torch.Tensor | None = None, wt: torch.Tensor | None = None, weights: str = "softmax",
               bias: torch.Tensor | None = None, groups: tuple | None = None) -> None:
@@ -788,25 +805,14 @@ def moe_route(z: torch.Tensor, n_experts: int, top: int, has_gate, dense: torch.
     scores divided by their sum (+ 1e-20).  groups (count, keep): the experts stand in `count` equal runs, only experts of
     the `keep` runs with the best single expert can be chosen."""
     _dev(z, dense, tok_seq, idx, wt, bias)
-    if bias is not None:
-        _f32c(bias, "bias")
-        if weights != "sigmoid" or bias.numel() != n_experts:
-            raise KernelError("moe_route: a choice bias needs sigmoid weights and one value per expert")
+    gate, n_groups, keep = _route_arguments(n_experts, top, has_gate, weights, bias, groups)
     _i32(tok_seq, "tok_seq")
     _f32c(dense, "dense")
     T = z.shape[0]
     W = n_experts + int(bool(has_gate))
-    gate = 2 if has_gate == "one" else int(bool(has_gate))
-    if weights not in _ROUTE_MODES:
-        raise KernelError(f"moe_route: weights must be one of {', '.join(_ROUTE_MODES)}, got {weights!r}")
-    n_groups, keep = groups or (0, 0)
-    if groups and (n_groups < 1 or n_experts % n_groups or not 1 <= keep <= n_groups or top > keep * (n_experts // n_groups)):
-        raise KernelError(f"moe_route: {n_experts} experts in {n_groups} groups of which {keep} stay cannot give {top}")
     if z.dtype != torch.float32 or z.stride(1) != 1 or z.shape[1] < (n_experts if gate == 2 else W) \
             or tuple(dense.shape) != (T, W):
         raise KernelError("moe_route: z float32 [T, >= E (+1)] and dense [T, E (+1)] expected")
-    if top > n_experts:
-        raise KernelError("moe_route: more experts chosen than there are")
     if idx is not None:
         _i32(idx, "idx")
     if wt is not None:
@@ -816,6 +822,30 @@ def moe_route(z: torch.Tensor, n_experts: int, top: int, has_gate, dense: torch.
             raise KernelError("moe_route: idx and wt must be [T, top]")
     _check(_fn("moe", "oe_moe_route")(_ptr(z), z.stride(0), n_experts, top, gate, _ROUTE_MODES[weights], _ptr(idx), _ptr(wt),
                                       _ptr(dense), _ptr(tok_seq), T, _ptr(bias), int(n_groups), int(keep), _stream()), "moe_route")
+
+
+def moe_router_supported(h: torch.Tensor, w: torch.Tensor) -> bool:
+    """Whether the kernel that makes the router's logits and routes by them takes these operands."""
+    return (h.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[0] <= 64 and w.shape[1] % 8 == 0
+            and w.is_contiguous() and h.stride(1) == 1 and h.stride(0) % 8 == 0 and h.data_ptr() % 16 == 0
+            and w.data_ptr() % 16 == 0)
+
+
+def moe_router(h: torch.Tensor, w: torch.Tensor, n_experts: int, top: int, has_gate, dense: torch.Tensor,
+               tok_seq: torch.Tensor, weights: str = "softmax", bias: torch.Tensor | None = None,
+               groups: tuple | None = None) -> None:
+    """moe_route on the logits h @ w.T (float32 sums), in one launch; h [T, D] and w [E (+ 1 with a gate), D] bfloat16."""
+    _dev(h, w, dense, tok_seq, bias)
+    gate, n_groups, keep = _route_arguments(n_experts, top, has_gate, weights, bias, groups)
+    _i32(tok_seq, "tok_seq")
+    _f32c(dense, "dense")
+    rows = n_experts + int(gate == 1)
+    if not moe_router_supported(h, w) or tuple(w.shape) != (rows, h.shape[1]) or tok_seq.numel() < h.shape[0] \
+            or tuple(dense.shape) != (h.shape[0], n_experts + int(gate > 0)):
+        raise KernelError("moe_router: h bfloat16 [T, D], w bfloat16 [E (+1), D] and dense [T, E (+1)] expected")
+    _check(_fn("moe", "oe_moe_router")(_ptr(h), h.stride(0), _ptr(w), h.shape[1], n_experts, top, gate, _ROUTE_MODES[weights],
+                                       _ptr(dense), _ptr(tok_seq), h.shape[0], _ptr(bias), n_groups, keep, _stream()),
+           "moe_router")
 
 
 def moe_dense_relu2(u: torch.Tensor, dense: torch.Tensor, ff: int) -> None:

@@ -34,6 +34,17 @@ from .registry import FEED_FORWARDS, Part
 from .spec import TensorDecl
 
 
+def _route(rt, h, w_route, experts: int, top: int, has_gate, dense, ctx, weights, bias, groups) -> None:
+    """`dense` from h through the router: one launch where the kernel takes the operands, else a product and the routing.
+    float32 sums and logits on both ways and both paths."""
+    if rt.tensor_cores and ops.moe_router_supported(h, w_route):
+        ops.moe_router(h, w_route, experts, top, has_gate, dense, ctx.tok_seq, weights, bias, groups)
+        return
+    z = rt.buffer("moe.z", h.shape[0], w_route.shape[0], dtype=torch.float32)
+    matmul_nt(rt, z, h, w_route)
+    ops.moe_route(z, experts, top, has_gate, dense, ctx.tok_seq, weights=weights, bias=bias, groups=groups)
+
+
 def _groups(raw, experts: int, top: int):
     """(count, keep) of a choice by groups, or None."""
     if not raw:
@@ -133,11 +144,9 @@ class MoESwiGLU(Part):
     def forward(self, h, residual, ctx, overwrite: bool = False):
         """overwrite: the output is written into `residual` (float32) instead of added."""
         T = h.shape[0]
-        z = self.rt.buffer("moe.z", T, self.w_route_rows(), dtype=torch.float32)
-        matmul_nt(self.rt, z, h, self.w_route)                  # float32 sums and output on both paths
         dense = self.rt.buffer("moe.dense", T, self.E + (1 if self.sff else 0), dtype=torch.float32)
-        ops.moe_route(z, self.E, self.top, (True if self.shared_gate else "one") if self.sff else False, dense,
-                      ctx.tok_seq, weights=self.router_weights, bias=self.bias, groups=self.groups)
+        _route(self.rt, h, self.w_route, self.E, self.top, (True if self.shared_gate else "one") if self.sff else False,
+               dense, ctx, self.router_weights, self.bias, self.groups)
         gu = self.rt.buffer("moe.gu", T, 2 * self.F)
         matmul_nt(self.rt, gu, h, self.w_gu)
         a = self.rt.buffer("moe.a", T, self.F)
@@ -198,10 +207,8 @@ class MoEReLU2(Part):
         """The routing, and what the up product does with its sums: squared ReLU times the token's weight for the
         column's expert (zero where it was not chosen)."""
         T = h.shape[0]
-        z = self.rt.buffer("moe.z", T, self.E, dtype=torch.float32)
-        matmul_nt(self.rt, z, h, self.w_route)                  # float32 sums and output on both paths
         dense = self.rt.buffer("moe.dense", T, self.E, dtype=torch.float32)
-        ops.moe_route(z, self.E, self.top, False, dense, ctx.tok_seq, weights=self.router_weights, groups=self.groups)
+        _route(self.rt, h, self.w_route, self.E, self.top, False, dense, ctx, self.router_weights, None, self.groups)
         return "relu2", (dense, self.ff)
 
     def forward(self, h, residual, ctx, overwrite: bool = False, projected=None):

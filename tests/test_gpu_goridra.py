@@ -144,6 +144,36 @@ def test_routing_kernel(E, top, groups):
         ops.moe_route(z.cuda(), E, top, False, dense, seq.cuda(), weights="softmax_all", groups=(E, 0))
 
 
+@pytest.mark.parametrize("T", [1, 7, 300, 1025])
+@pytest.mark.parametrize("E,top,groups,gate,weights", [(8, 2, (4, 2), False, "softmax_all"), (5, 1, None, False, "softmax_all"),
+                                                       (7, 3, None, True, "softmax"), (16, 4, (8, 4), False, "softmax_all"),
+                                                       (12, 2, None, "one", "sigmoid"), (31, 3, None, True, "softmax"),
+                                                       (64, 6, (16, 3), False, "softmax_all")])
+@pytest.mark.parametrize("D", [64, 2056])
+def test_router_in_one_launch(T, E, top, groups, gate, weights, D):
+    """The router's product and the routing in one launch against the routing kernel on float64 logits: the same choice
+    wherever it is no close call, whatever else is in the batch."""
+    from oracle_engine_b200.csrc import ops
+    g = torch.Generator().manual_seed(T + E + D)
+    rows = E + (1 if gate is True else 0)
+    wide = torch.randn(T, D + 8, generator=g).bfloat16().cuda()
+    h, w = wide[:, :D], (torch.randn(rows, D, generator=g) * 2 / D ** 0.5).bfloat16().cuda()
+    seq = torch.zeros(T, dtype=torch.int32)
+    if T > 5:
+        seq[4] = -1
+    bias = torch.randn(E, generator=g).cuda() * 0.1 if weights == "sigmoid" else None
+    z = h.double() @ w.double().T
+    want, got = (torch.full((T, E + int(bool(gate))), 9.0, device="cuda") for _ in range(2))
+    ops.moe_route(z.float().contiguous(), E, top, gate, want, seq.cuda(), weights=weights, bias=bias, groups=groups)
+    ops.moe_router(h, w, E, top, gate, got, seq.cuda(), weights, bias, groups)
+    same = ((got > 0) == (want > 0)).all(1)
+    assert same.float().mean().item() > 0.99 or (~same).sum().item() <= 1
+    assert (got[same] - want[same]).abs().max().item() < 2e-5
+    last = torch.full((1, got.shape[1]), 9.0, device="cuda")                     # the last token alone: the same bits
+    ops.moe_router(h[-1:], w, E, top, gate, last, torch.zeros(1, dtype=torch.int32).cuda(), weights, bias, groups)
+    assert torch.equal(last[0], got[-1])
+
+
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("ff", [24, 10])
 def test_squared_relu_experts_kernel(dtype, ff):
