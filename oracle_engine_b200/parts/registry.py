@@ -30,6 +30,10 @@ Mixer  (MIXERS; e.g. attention)
     times the constant m and the float32 per-channel vector s, or None, is added): arrangements that norm or
     scale what a sublayer returns ask for these and fall back to a buffer of their own
 
+    optional: parts with `joint_weight` (the attribute that holds the first matrix) whose forward takes `projected=`, a
+    feed-forward also with `joint_epilogue(h, ctx)`, can have their first products computed as one by an arrangement
+    that gives both the same input (parts/block.py: JoinedInput)
+
 FeedForward  (FEED_FORWARDS; dense or routed)
     forward(h, residual, ctx)            adds its output into residual
 
