@@ -11,6 +11,11 @@
 //   unrotate_heads       every head of o [T, H dv] turned back by its own token's position (angle -pos * f_m), in place:
 //                        with values stored turned by the key's position, a softmax-weighted sum turned back by the
 //                        query's position depends on the values through relative positions only.
+//   qkv_row_norm_rot_write   one block per token of the row [q: H dk | k: G dk | v: G dv | ...] (float32 or bfloat16): q
+//                        divided by the root mean square of ALL its H dk values and times a weight of that size, k likewise
+//                        over its G dk values (the norm may be absent); then the first `rot` dimensions of every head
+//                        turned by the token's position, 2i paired with 2i + 1 or i with i + rot/2.  q goes back in place, k
+//                        and v to the token's cache rows.
 // All arithmetic is float32.
 #include "common.cuh"
 
@@ -104,6 +109,78 @@ qkv_norm_rot_write_kernel(T* q_out, T* kcache, T* vcache, const PrepArgs a) {
     }
 }
 
+struct RowPrepArgs {
+    long long ld;
+    const float* qw; const float* kw; float eps;
+    const float* cos_t; const float* sin_t; int rot, halves;
+    const int* tables; int max_pages;
+    const int* tok_seq; const int* tok_pos;
+    int n_tokens, H, G, dk, dv;
+};
+
+constexpr int ROW_THREADS = 256;
+
+// A turned pair of head values: where its two values lie behind the first column of the head.
+__device__ __forceinline__ void pair_columns(int i, int rot, int halves, int& first, int& second) {
+    if (halves) { first = i; second = i + rot / 2; }
+    else { first = 2 * i; second = 2 * i + 1; }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(ROW_THREADS)
+qkv_row_norm_rot_write_kernel(T* qkv, T* kcache, T* vcache, const RowPrepArgs a) {
+    __shared__ float red[2][32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int b = a.tok_seq[t];
+    if (b < 0) return;
+    const int pos = a.tok_pos[t];
+    const int page = a.tables[(size_t)b * a.max_pages + pos / OE_PAGE];
+    T* row = qkv + (size_t)t * a.ld;
+    const int qn = a.H * a.dk, kn = a.G * a.dk, vn = a.G * a.dv;
+    T* krow = row + qn;
+    const T* vrow = krow + kn;
+    float sq = 1.f, sk = 1.f;
+    if (a.qw) {
+        float s = 0.f, u = 0.f;
+        for (int i = threadIdx.x; i < qn; i += ROW_THREADS) { const float v = to_f32(row[i]); s = fmaf(v, v, s); }
+        for (int i = threadIdx.x; i < kn; i += ROW_THREADS) { const float v = to_f32(krow[i]); u = fmaf(v, v, u); }
+        s = block_sum(s, red[0]);
+        u = block_sum(u, red[1]);
+        sq = 1.f / sqrtf(s / (float)qn + a.eps);
+        sk = 1.f / sqrtf(u / (float)kn + a.eps);
+    }
+    const int half = a.rot / 2;
+    const float* cr = a.cos_t + (size_t)pos * half;
+    const float* sr = a.sin_t + (size_t)pos * half;
+    const int rest = a.dk - half;                 // what a head takes: `half` pairs, then the dimensions that pass
+    // q and k heads: a thread owns whole pairs, so that it may write where it read
+    for (int e = threadIdx.x; e < (a.H + a.G) * rest; e += ROW_THREADS) {
+        const int hh = e / rest, i = e % rest;
+        const bool key = hh >= a.H;
+        const int head = key ? hh - a.H : hh;
+        if (key && page < 0) continue;
+        const T* src = (key ? krow : row) + (size_t)head * a.dk;
+        T* dst = key ? kcache + (((size_t)page * a.G + head) * OE_PAGE + (pos % OE_PAGE)) * a.dk : row + (size_t)head * a.dk;
+        const float* w = a.qw ? (key ? a.kw : a.qw) + (size_t)head * a.dk : nullptr;
+        const float s = key ? sk : sq;
+        if (i < half) {
+            int c0, c1;
+            pair_columns(i, a.rot, a.halves, c0, c1);
+            const float u = to_f32(src[c0]) * s * (w ? w[c0] : 1.f), v = to_f32(src[c1]) * s * (w ? w[c1] : 1.f);
+            dst[c0] = from_f32<T>(u * cr[i] - v * sr[i]);
+            dst[c1] = from_f32<T>(v * cr[i] + u * sr[i]);
+        } else {
+            const int c = i + half;
+            dst[c] = from_f32<T>(to_f32(src[c]) * s * (w ? w[c] : 1.f));
+        }
+    }
+    if (page < 0) return;
+    for (int e = threadIdx.x; e < vn; e += ROW_THREADS)
+        vcache[(((size_t)page * a.G + e / a.dv) * OE_PAGE + (pos % OE_PAGE)) * a.dv + e % a.dv] = vrow[e];
+}
+
 template <typename T>
 __global__ void __launch_bounds__(WARPS * 32)
 unrotate_heads_kernel(T* o, const float* __restrict__ cos_v, const float* __restrict__ sin_v,
@@ -141,6 +218,21 @@ int launch_prep(T* q_out, T* kcache, T* vcache, const PrepArgs& a, cudaStream_t 
     const long long blocks = (items + WARPS - 1) / WARPS;
     if (blocks > 2147483647LL) return OE_ERR_UNSUPPORTED;
     return oe_launch(qkv_norm_rot_write_kernel<T>, dim3((unsigned)blocks), dim3(WARPS * 32), 0, st, q_out, kcache, vcache, a);
+}
+
+template <typename T>
+int launch_row_prep(T* qkv, long long ld, T* kcache, T* vcache, const float* qw, const float* kw, float eps, const float* cos_t,
+                    const float* sin_t, int rot, int halves, const int* tables, int max_pages, const int* tok_seq,
+                    const int* tok_pos, int n_tokens, int H, int G, int dk, int dv, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
+    if (H < 1 || G < 1 || dk < 1 || dv < 1 || rot < 0 || rot % 2 || rot > dk || (qw == nullptr) != (kw == nullptr) ||
+        (rot && (cos_t == nullptr || sin_t == nullptr)))
+        return OE_ERR_UNSUPPORTED;
+    RowPrepArgs a;
+    a.ld = ld; a.qw = qw; a.kw = kw; a.eps = eps; a.cos_t = cos_t; a.sin_t = sin_t; a.rot = rot; a.halves = halves;
+    a.tables = tables; a.max_pages = max_pages; a.tok_seq = tok_seq; a.tok_pos = tok_pos;
+    a.n_tokens = n_tokens; a.H = H; a.G = G; a.dk = dk; a.dv = dv;
+    return oe_launch(qkv_row_norm_rot_write_kernel<T>, dim3(n_tokens), dim3(ROW_THREADS), 0, st, qkv, kcache, vcache, a);
 }
 
 template <typename T>
@@ -185,6 +277,20 @@ int oe_qkv_norm_rot_write_bf16(bf16* q_out, bf16* kcache, bf16* vcache, const fl
                                int n_tokens, int H, int G, int dk, int dv, cudaStream_t st) {
     return launch_prep<bf16>(q_out, kcache, vcache, make_args(proj, ld, qb, kb, vb, qw, kw, eps, cos_k, sin_k, rot, cos_v, sin_v,
                                                               v_norm, tables, max_pages, tok_seq, tok_pos, n_tokens, H, G, dk, dv), st);
+}
+int oe_qkv_row_norm_rot_write_f32(float* qkv, long long ld, float* kcache, float* vcache, const float* qw, const float* kw,
+                                  float eps, const float* cos_t, const float* sin_t, int rot, int halves, const int* tables,
+                                  int max_pages, const int* tok_seq, const int* tok_pos, int n_tokens, int H, int G, int dk,
+                                  int dv, cudaStream_t st) {
+    return launch_row_prep<float>(qkv, ld, kcache, vcache, qw, kw, eps, cos_t, sin_t, rot, halves, tables, max_pages, tok_seq,
+                                  tok_pos, n_tokens, H, G, dk, dv, st);
+}
+int oe_qkv_row_norm_rot_write_bf16(bf16* qkv, long long ld, bf16* kcache, bf16* vcache, const float* qw, const float* kw,
+                                   float eps, const float* cos_t, const float* sin_t, int rot, int halves, const int* tables,
+                                   int max_pages, const int* tok_seq, const int* tok_pos, int n_tokens, int H, int G, int dk,
+                                   int dv, cudaStream_t st) {
+    return launch_row_prep<bf16>(qkv, ld, kcache, vcache, qw, kw, eps, cos_t, sin_t, rot, halves, tables, max_pages, tok_seq,
+                                 tok_pos, n_tokens, H, G, dk, dv, st);
 }
 int oe_unrotate_heads_f32(float* o, const float* cos_v, const float* sin_v, const int* tok_seq, const int* tok_pos,
                           int n_tokens, int H, int dv, cudaStream_t st) {

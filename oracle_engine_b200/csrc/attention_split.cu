@@ -14,7 +14,9 @@
 //                         kernel (attention_split_mma.cu) does not take.  `sinks` (null, or one float32 per query
 //                         head): the softmax's denominator also holds exp(sinks[h]), a term without key or value.
 //                         `unrot_cos`, `unrot_sin` (null, or float32 [positions, dv/2]): every head's result is turned
-//                         back by its query's position, pair (m, m + dv/2), before it is stored.
+//                         back by its query's position, pair (m, m + dv/2), before it is stored.  `gate` (gate_mode
+//                         OE_GATE_VALUE: rows of one value per result, OE_GATE_HEAD: one per head; strides free): the
+//                         result is multiplied by the gate's sigmoid where it is stored.
 #include "common.cuh"
 
 namespace {
@@ -84,7 +86,7 @@ attn_split_kernel(T* out, const T* q, long long q_stride, const T* kcache, const
                   const int* __restrict__ tables, int max_pages, const int* __restrict__ tok_seq,
                   const int* __restrict__ tok_pos, int n_tokens, int H, int G, int dk, int dv, int window, float scale,
                   float cap, const float* __restrict__ sinks, const float* __restrict__ unrot_cos,
-                  const float* __restrict__ unrot_sin) {
+                  const float* __restrict__ unrot_sin, const T* gate, long long gate_stride, int gate_mode) {
     extern __shared__ float qs_all[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_launch_dependents();
@@ -165,6 +167,7 @@ attn_split_kernel(T* out, const T* q, long long q_stride, const T* kcache, const
             float r = qs[d];
             if (d < half) r = qs[d] * cr[d] + qs[d + half] * sr[d];
             else if (d < 2 * half) r = qs[d] * cr[d - half] - qs[d - half] * sr[d - half];
+            if (gate_mode) r *= oe_sigmoid_gate(gate, gate_stride, gate_mode, t, h, H, dv, d);
             o[d] = from_f32<T>(r);
         }
         return;
@@ -172,7 +175,10 @@ attn_split_kernel(T* out, const T* q, long long q_stride, const T* kcache, const
 #pragma unroll
     for (int i = 0; i < MAX_D / 32; i++) {
         const int d = lane + 32 * i;
-        if (d < dv) o[d] = from_f32<T>(acc[i] * inv);
+        if (d >= dv) continue;
+        float r = acc[i] * inv;
+        if (gate_mode) r *= oe_sigmoid_gate(gate, gate_stride, gate_mode, t, h, H, dv, d);
+        o[d] = from_f32<T>(r);
     }
 }
 
@@ -195,8 +201,9 @@ template <typename T>
 int launch_attn(T* out, const T* q, long long q_stride, const T* kcache, const T* vcache, const int* tables,
                 int max_pages, const int* tok_seq, const int* tok_pos, int n_tokens, int H, int G, int dk, int dv,
                 int window, float scale, float cap, const float* sinks, const float* unrot_cos, const float* unrot_sin,
-                cudaStream_t st) {
+                const T* gate, long long gate_stride, int gate_mode, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
+    if (gate_mode < 0 || gate_mode > OE_GATE_HEAD || (gate_mode && gate == nullptr)) return OE_ERR_UNSUPPORTED;
     if (unrot_cos == nullptr || unrot_sin == nullptr) unrot_cos = unrot_sin = nullptr;
     if (dk < 1 || dk > MAX_D || dv < 1 || dv > MAX_D || G < 1 || H % G) return OE_ERR_UNSUPPORTED;
     const long long items = (long long)n_tokens * H;
@@ -204,7 +211,7 @@ int launch_attn(T* out, const T* q, long long q_stride, const T* kcache, const T
     if (blocks > 2147483647LL) return OE_ERR_UNSUPPORTED;
     return oe_launch(attn_split_kernel<T>, dim3((unsigned)blocks), dim3(WARPS * 32), WARPS * (dk > dv ? dk : dv) * sizeof(float), st, out, q,
                      q_stride, kcache, vcache, tables, max_pages, tok_seq, tok_pos, n_tokens, H, G, dk, dv, window, scale,
-                     cap, sinks, unrot_cos, unrot_sin);
+                     cap, sinks, unrot_cos, unrot_sin, gate, gate_stride, gate_mode);
 }
 
 }  // namespace
@@ -227,15 +234,17 @@ int oe_rope_split_kv_write_bf16(bf16* qkv, long long stride, const float* cos_t,
 int oe_attn_split_f32(float* out, const float* q, long long q_stride, const float* kcache, const float* vcache,
                       const int* tables, int max_pages, const int* tok_seq, const int* tok_pos, int n_tokens, int H,
                       int G, int dk, int dv, int window, float scale, float cap, const float* sinks,
-                      const float* unrot_cos, const float* unrot_sin, cudaStream_t st) {
+                      const float* unrot_cos, const float* unrot_sin, const float* gate, long long gate_stride,
+                      int gate_mode, cudaStream_t st) {
     return launch_attn<float>(out, q, q_stride, kcache, vcache, tables, max_pages, tok_seq, tok_pos, n_tokens, H, G, dk,
-                              dv, window, scale, cap, sinks, unrot_cos, unrot_sin, st);
+                              dv, window, scale, cap, sinks, unrot_cos, unrot_sin, gate, gate_stride, gate_mode, st);
 }
 int oe_attn_split_bf16(bf16* out, const bf16* q, long long q_stride, const bf16* kcache, const bf16* vcache,
                        const int* tables, int max_pages, const int* tok_seq, const int* tok_pos, int n_tokens, int H,
                        int G, int dk, int dv, int window, float scale, float cap, const float* sinks,
-                       const float* unrot_cos, const float* unrot_sin, cudaStream_t st) {
+                       const float* unrot_cos, const float* unrot_sin, const bf16* gate, long long gate_stride,
+                       int gate_mode, cudaStream_t st) {
     return launch_attn<bf16>(out, q, q_stride, kcache, vcache, tables, max_pages, tok_seq, tok_pos, n_tokens, H, G, dk,
-                             dv, window, scale, cap, sinks, unrot_cos, unrot_sin, st);
+                             dv, window, scale, cap, sinks, unrot_cos, unrot_sin, gate, gate_stride, gate_mode, st);
 }
 }

@@ -14,6 +14,8 @@
 // A step of single tokens may split a sequence's pages over `n_splits` CTAs (grid x): each writes its unnormalised
 // sums, maximum and denominator as float32, and attn_split_merge_kernel puts them together in split order.
 //
+// An output gate multiplies the result by its sigmoid where it is stored (here or in the merge).
+//
 // -DOE_KV_SHARED=1: the values are the first DV columns of the key rows (DV <= DK), one tensor [pages][KVH][64][DK]:
 // attention over a cache of latents, where a row [latent | shared key part] is the key of every head and its first
 // part the value (csrc/attention_latent.cu).  Only the key panel is staged; P V reads its first DV columns.
@@ -60,6 +62,9 @@ struct Args {
     const float* sinks;        // null, or [H] float32: exp(sinks[h]) joins the softmax's denominator (no key, no value)
     const float* unrot_cos;    // null, or [positions, DV/2] float32 (with unrot_sin): every head's result is turned back by
     const float* unrot_sin;    //   its query's position, pair (m, m + DV/2) by minus the table's angle, before it is stored
+    const bf16* gate;          // rows of gate_stride elements (even, 4-byte aligned for OE_GATE_VALUE), or null
+    long long gate_stride;
+    int gate_mode;             // 0 none, OE_GATE_VALUE, OE_GATE_HEAD: the stored result is multiplied by the gate's sigmoid
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
@@ -303,7 +308,9 @@ attn_split_mma_kernel(const Args a) {
 #pragma unroll
     for (int i = 0; i < 2; i++) {
         if (!valid[i]) continue;
-        const float inv = l_run[i] > 0.f ? 1.f / l_run[i] : 0.f;
+        float inv = l_run[i] > 0.f ? 1.f / l_run[i] : 0.f;
+        const bf16* gr = a.gate + (packed0 + tok[i]) * a.gate_stride;
+        if (a.gate_mode == OE_GATE_HEAD) inv *= oe_sigmoid(__bfloat162float(gr[head[i]]));
         bf16* o = a.out + (packed0 + tok[i]) * (long long)(a.H * DV) + (size_t)head[i] * DV + tig * 2;
         if (a.unrot_cos != nullptr) {
             // column m of the first half and m + DV/2 lie in the same thread: accumulators n and n + DV/16
@@ -319,6 +326,15 @@ attn_split_mma_kernel(const Args a) {
             }
             continue;
         }
+        if (a.gate_mode == OE_GATE_VALUE) {
+            gr += (size_t)head[i] * DV + tig * 2;
+#pragma unroll
+            for (int n = 0; n < DV / 8; n++) {
+                const float2 g = __bfloat1622float2(*(const __nv_bfloat162*)(gr + n * 8));
+                *(uint32_t*)(o + n * 8) = pack_bf16(oacc[n][2 * i] * inv * oe_sigmoid(g.x), oacc[n][2 * i + 1] * inv * oe_sigmoid(g.y));
+            }
+            continue;
+        }
 #pragma unroll
         for (int n = 0; n < DV / 8; n++)
             *(uint32_t*)(o + n * 8) = pack_bf16(oacc[n][2 * i] * inv, oacc[n][2 * i + 1] * inv);
@@ -329,7 +345,8 @@ attn_split_mma_kernel(const Args a) {
 __global__ void __launch_bounds__(128)
 attn_split_merge_kernel(bf16* out, const float* partial, int n_splits, const int* __restrict__ seq_qlen, int H,
                         const float* __restrict__ sinks, const float* __restrict__ unrot_cos,
-                        const float* __restrict__ unrot_sin, const int* __restrict__ seq_start) {
+                        const float* __restrict__ unrot_sin, const int* __restrict__ seq_start, const bf16* gate,
+                        long long gate_stride, int gate_mode) {
     pdl_launch_dependents();
     pdl_wait();
     if (seq_qlen[blockIdx.x / H] <= 0) {                 // a padding sequence: nothing was written for it
@@ -346,7 +363,9 @@ attn_split_merge_kernel(bf16* out, const float* partial, int n_splits, const int
         const float ms = p[(size_t)s * (DV + 2) + DV];
         if (ms != -INFINITY) l += exp2f(ms - m) * p[(size_t)s * (DV + 2) + DV + 1];
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    const int gt = blockIdx.x / H, gh = blockIdx.x % H;          // token and head
+    if (gate_mode == OE_GATE_HEAD) inv *= oe_sigmoid_gate(gate, gate_stride, gate_mode, gt, gh, H, DV, 0);
     if (unrot_cos != nullptr) {
         // the sequence's one token stands at position seq_start; a thread takes a pair (d, d + DV/2) and turns it back
         const size_t at = (size_t)seq_start[blockIdx.x / H] * (DV / 2);
@@ -374,7 +393,9 @@ attn_split_merge_kernel(bf16* out, const float* partial, int n_splits, const int
             const float ms = p[(size_t)s * (DV + 2) + DV];
             if (ms != -INFINITY) acc = fmaf(exp2f(ms - m), p[(size_t)s * (DV + 2) + d], acc);
         }
-        out[(size_t)blockIdx.x * DV + d] = __float2bfloat16_rn(acc * inv);
+        acc *= inv;
+        if (gate_mode == OE_GATE_VALUE) acc *= oe_sigmoid_gate(gate, gate_stride, gate_mode, gt, gh, H, DV, d);
+        out[(size_t)blockIdx.x * DV + d] = __float2bfloat16_rn(acc);
     }
 }
 
@@ -388,7 +409,8 @@ int oe_attn_split_mma_dims(int* dk, int* dv) { *dk = DK; *dv = DV; return 0; }
 int oe_attn_split_mma(bf16* out, const bf16* q, long long q_stride, const bf16* kcache, const bf16* vcache,
                       const int* tables, int max_pages, const int* cu_q, const int* seq_start, const int* seq_qlen,
                       int n_seqs, int max_qlen, int H, int KVH, int window, float scale, float cap, int n_splits,
-                      float* partial, const float* sinks, const float* unrot_cos, const float* unrot_sin, cudaStream_t st) {
+                      float* partial, const float* sinks, const float* unrot_cos, const float* unrot_sin, const bf16* gate,
+                      long long gate_stride, int gate_mode, cudaStream_t st) {
     if (n_seqs <= 0 || max_qlen <= 0) return 0;
     if (KVH < 1 || H % KVH || H / KVH > NWARPS * 16 || n_seqs > 65535 || KVH > 65535) return OE_ERR_UNSUPPORTED;
     if (n_splits > 1 && (max_qlen != 1 || partial == nullptr)) return OE_ERR_UNSUPPORTED;
@@ -401,6 +423,9 @@ int oe_attn_split_mma(bf16* out, const bf16* q, long long q_stride, const bf16* 
     a.partial = partial;
     a.sinks = sinks;
     const bool unrot = unrot_cos != nullptr && unrot_sin != nullptr;
+    if (gate_mode < 0 || gate_mode > OE_GATE_HEAD || (gate_mode && gate == nullptr) || (gate_mode == OE_GATE_VALUE && unrot))
+        return OE_ERR_UNSUPPORTED;
+    a.gate = gate; a.gate_stride = gate_stride; a.gate_mode = gate_mode;
     // with several splits the merge turns the result back, not the kernel that writes the parts
     a.unrot_cos = unrot && a.n_splits <= 1 ? unrot_cos : nullptr;
     a.unrot_sin = unrot && a.n_splits <= 1 ? unrot_sin : nullptr;
@@ -416,7 +441,8 @@ int oe_attn_split_mma(bf16* out, const bf16* q, long long q_stride, const bf16* 
         const int rc = oe_launch(attn_split_mma_kernel, dim3(a.n_splits, KVH, n_seqs), dim3(NWARPS * 32), smem, st, a);
         if (rc) return rc;
         return oe_launch(attn_split_merge_kernel, dim3(n_seqs * H), dim3(128), 0, st, out, (const float*)partial, a.n_splits, seq_qlen, H, sinks,
-                         unrot ? unrot_cos : (const float*)nullptr, unrot ? unrot_sin : (const float*)nullptr, seq_start);
+                         unrot ? unrot_cos : (const float*)nullptr, unrot ? unrot_sin : (const float*)nullptr, seq_start,
+                         gate, gate_stride, gate_mode);
     }
     const dim3 grid((max_qlen + a.tokens_per_tile - 1) / a.tokens_per_tile, KVH, n_seqs);
     return oe_launch(attn_split_mma_kernel, grid, dim3(NWARPS * 32), smem, st, a);

@@ -45,6 +45,7 @@ LIBRARIES = {
     "tokenwise": ("tokenwise.cu", []),
     "attention_prep": ("attention_prep.cu", []),
     "general_delta": ("general_delta.cu", []),
+    "selective_scan": ("selective_scan.cu", []),
     "gemm_tc": ("gemm_tcgen05.cu", []),
     "gemm_pair": ("gemm_tcgen05_pair.cu", []),
     "gemm_skinny": ("gemm_skinny.cu", []),

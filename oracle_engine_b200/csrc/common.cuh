@@ -115,6 +115,16 @@ template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
+// An output gate of an attention: what head h's result of token t is multiplied by at column d, sigmoid of the row's value
+// for that column (OE_GATE_VALUE, rows of H dv values) or of the head's value (OE_GATE_HEAD, rows of H values).
+#define OE_GATE_VALUE 1
+#define OE_GATE_HEAD 2
+__device__ __forceinline__ float oe_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+template <typename T>
+__device__ __forceinline__ float oe_sigmoid_gate(const T* gate, long long stride, int mode, long long t, int h, int H, int dv, int d) {
+    return oe_sigmoid(to_f32(gate[t * stride + (mode == OE_GATE_HEAD ? h : (long long)h * dv + d)]));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

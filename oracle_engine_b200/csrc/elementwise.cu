@@ -14,7 +14,7 @@
 // ---------------------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_gather_kernel(float* __restrict__ x, const T* __restrict__ table,
-                                    const int* __restrict__ ids, int D, int vocab, int* err) {
+                                    const int* __restrict__ ids, int D, int vocab, float scale, int* err) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -26,7 +26,7 @@ __global__ void embed_gather_kernel(float* __restrict__ x, const T* __restrict__
         return;
     }
     const T* row = table + (size_t)id * D;
-    for (int d = threadIdx.x; d < D; d += blockDim.x) xr[d] = to_f32(row[d]);
+    for (int d = threadIdx.x; d < D; d += blockDim.x) xr[d] = to_f32(row[d]) * scale;
 }
 
 // ---------------------------------------------------------------------------------------
@@ -540,15 +540,15 @@ __global__ void gather_rows_f32_kernel(float* out, const float* x,
 extern "C" {
 
 int oe_embed_gather_f32(float* x, const float* table, const int* ids, int n_tokens, int D, int vocab,
-                        int* err, cudaStream_t st) {
+                        float scale, int* err, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
-    const int launch_rc = oe_launch(embed_gather_kernel<float>, dim3(n_tokens), dim3(256), 0, st, x, table, ids, D, vocab, err);
+    const int launch_rc = oe_launch(embed_gather_kernel<float>, dim3(n_tokens), dim3(256), 0, st, x, table, ids, D, vocab, scale, err);
     return launch_rc;
 }
 int oe_embed_gather_bf16(float* x, const bf16* table, const int* ids, int n_tokens, int D, int vocab,
-                         int* err, cudaStream_t st) {
+                         float scale, int* err, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
-    const int launch_rc = oe_launch(embed_gather_kernel<bf16>, dim3(n_tokens), dim3(256), 0, st, x, table, ids, D, vocab, err);
+    const int launch_rc = oe_launch(embed_gather_kernel<bf16>, dim3(n_tokens), dim3(256), 0, st, x, table, ids, D, vocab, scale, err);
     return launch_rc;
 }
 

@@ -8,7 +8,8 @@
 //                   in the last column sigmoid(gate logit) (has_gate 1) or one (has_gate 2: a shared expert without
 //                   a gate; z then holds no column for it).  mode 1: the weight of a chosen expert is the sigmoid
 //                   of its own logit, not renormalised (the choice is by the same order).  With `bias` (one float32
-//                   per expert, mode 1 only) the choice is by sigmoid(z) + bias and the weight stays sigmoid(z).
+//                   per expert) in mode 1 the choice is by sigmoid(z) + bias and the weight stays sigmoid(z); in modes 0
+//                   and 2 the bias is part of the logits: choice and weights are those of z + bias.
 //                   mode 2: the scores are the softmax over ALL experts, the weights the chosen scores over (their sum
 //                   + 1e-20).  n_groups > 0: the experts stand in n_groups equal runs, a run's score is its best
 //                   expert's, and only experts of the `keep` best runs can be chosen.
@@ -40,7 +41,10 @@ __device__ __forceinline__ void route_token(const float* zr, int t, int lane, in
     }
     __syncwarp();
     // what the choice goes by: a logit (its order is the softmax's), or sigmoid + bias
-    auto score = [&](int e) { return bias ? 1.f / (1.f + expf(-zr[e])) + bias[e] : zr[e]; };
+    auto score = [&](int e) {
+        if (!bias) return zr[e];
+        return (mode == 1 ? 1.f / (1.f + expf(-zr[e])) : zr[e]) + bias[e];
+    };
     const int per_run = n_groups > 0 ? E / n_groups : E;
     if (n_groups > 0) {
         kept[lane] = 0u;
@@ -101,7 +105,7 @@ __device__ __forceinline__ void route_token(const float* zr, int t, int lane, in
         // zmax is the largest logit of all: the best run holds it.  With Z = sum_all exp(z - zmax) a score is
         // p / Z, and p / Z / (sum / Z + 1e-20) is the weight.
         float total = 0.f;
-        for (int e = lane; e < E; e += 32) total += expf(zr[e] - zmax);
+        for (int e = lane; e < E; e += 32) total += expf(score(e) - zmax);
         total = warp_sum(total);
         inv = 1.f / total / (sum / total + 1e-20f);
     }
@@ -305,7 +309,7 @@ extern "C" {
 int oe_moe_route(const float* z, long long ldz, int E, int top, int has_gate, int mode, int* idx, float* wt, float* dense,
                  const int* tok_seq, int n_tokens, const float* bias, int n_groups, int keep, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
-    if (E < 1 || E > 1024 || top < 1 || mode < 0 || mode > 2 || (bias != nullptr && mode != 1)) return OE_ERR_UNSUPPORTED;
+    if (E < 1 || E > 1024 || top < 1 || mode < 0 || mode > 2) return OE_ERR_UNSUPPORTED;
     if (n_groups < 0 || (n_groups > 0 && (E % n_groups || keep < 1 || keep > n_groups))) return OE_ERR_UNSUPPORTED;
     return oe_launch(moe_route_kernel, dim3((n_tokens + 3) / 4), dim3(128), 0, st, z, ldz, E, top, has_gate, mode, idx, wt, dense,
                      tok_seq, n_tokens, bias, n_groups, keep);
@@ -315,7 +319,7 @@ int oe_moe_router(const bf16* h, long long ldh, const bf16* w, int D, int E, int
                   const int* tok_seq, int n_tokens, const float* bias, int n_groups, int keep, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     const int R = E + (has_gate == 1 ? 1 : 0);
-    if (E < 1 || R > 64 || top < 1 || mode < 0 || mode > 2 || (bias != nullptr && mode != 1)) return OE_ERR_UNSUPPORTED;
+    if (E < 1 || R > 64 || top < 1 || mode < 0 || mode > 2) return OE_ERR_UNSUPPORTED;
     if (n_groups < 0 || (n_groups > 0 && (E % n_groups || keep < 1 || keep > n_groups))) return OE_ERR_UNSUPPORTED;
     if (D % 8 || ldh % 8 || (((uintptr_t)h | (uintptr_t)w) & 15)) return OE_ERR_UNSUPPORTED;
 #define OE_ROUTER(ROWS, TOK)                                                                                              \

@@ -33,7 +33,7 @@ _SUFFIX = {torch.float32: "f32", torch.bfloat16: "bf16"}
 _P, _I, _F, _L = c_void_p, c_int, c_float, c_longlong
 _SIGNATURES = {
     "elementwise": {
-        "oe_embed_gather": [_P, _P, _P, _I, _I, _I, _P, _P],
+        "oe_embed_gather": [_P, _P, _P, _I, _I, _I, _F, _P, _P],
         "oe_rmsnorm": [_P, _P, _P, _I, _I, _F, _P],
         "oe_layernorm": [_P, _P, _P, _P, _I, _I, _F, _P],
         "oe_rope_kv_write": [_P, _I, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
@@ -49,6 +49,7 @@ _SIGNATURES = {
     "rowwise": {
         "oe_cast_rows_bf16": [_P, _P, _L, _P],
         "oe_rmsnorm_add": [_P, _P, _P, _I, _I, _F, _F, _I, _P, _P],
+        "oe_rmsnorm_sum": [_P, _P, _P, _P, _P, _F, _F, _P, _I, _I, _F, _P, _P],
         "oe_relu2": [_P, _L, _P],
         "oe_gelu": [_P, _L, _P],
         "oe_tanh_rows": [_P, _P, _L, _P],
@@ -58,12 +59,13 @@ _SIGNATURES = {
     },
     "attention_split": {
         "oe_rope_split_kv_write": [_P, _L, _P, _P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-        "oe_attn_split": [_P, _P, _L, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P, _P, _P, _P],
+        "oe_attn_split": [_P, _P, _L, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P, _P, _P, _P, _L, _I, _P],
     },
     "attention_prep": {
         "oe_qkv_norm_rot_write": [_P, _P, _P, _P, _L, _P, _P, _P, _P, _P, _F, _P, _P, _I, _P, _P, _I, _P, _I, _P, _P,
                                   _I, _I, _I, _I, _I, _P],
         "oe_unrotate_heads": [_P, _P, _P, _P, _P, _I, _I, _I, _P],
+        "oe_qkv_row_norm_rot_write": [_P, _L, _P, _P, _P, _P, _F, _P, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
     },
     "tokenwise": {
         "oe_dyt_norm": [_P, _P, _P, _P, _F, _L, _I, _P],
@@ -77,6 +79,14 @@ _SIGNATURES = {
         "oe_gdelta_padded_dk": [_I],
         "oe_gdelta_prepare": [_P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _I, _I, _I, _P],
         "oe_gdelta_scan": [_P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _P],
+    },
+    "selective_scan": {
+        "oe_causal_conv": [_P, _P, _L, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P],
+        "oe_conv_rows_state": [_P, _P, _L, _I, _I, _P, _P, _I, _P],
+        "oe_thin_cast": [_P, _P, _L, _I, _I, _P],
+        "oe_selective_scan": [_P, _P, _P, _P, _P, _P, _L, _I, _I, _P, _P, _P, _L, _P, _P, _I, _I, _I, _P],
+        "oe_selective_scan_segments": [_P, _P, _P, _P, _P, _P, _L, _I, _I, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P],
+        "oe_selective_step": [_P, _P, _P, _P, _I, _I, _I, _P, _P, _L, _I, _I, _P, _P, _P, _L, _P, _P, _I, _I, _I, _P],
     },
     "retention": {
         "oe_retention_scan": [_P, _P, _P, _L, _I, _I, _I, _P, _P, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _P],
@@ -100,8 +110,8 @@ _SIGNATURES = {
         "oe_gla_scan_segments": [_P, _P, _P, _P, _P, _L, _P, _L, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _I, _P, _P, _P],
     },
     "attention_latent": {
-        "oe_latent_write": [_P, _L, _P, _F, _P, _L, _P, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-        "oe_attn_latent": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _P],
+        "oe_latent_write": [_P, _L, _P, _F, _P, _L, _P, _P, _P, _P, _I, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+        "oe_attn_latent": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P, _L, _P],
         "oe_head_matmul": [_P, _L, _L, _P, _L, _L, _P, _I, _I, _I, _I, _P],
     },
     "recurrent": {
@@ -122,7 +132,8 @@ _TYPED = {"oe_embed_gather", "oe_rmsnorm", "oe_rope_kv_write", "oe_swiglu", "oe_
           "oe_relu2", "oe_gelu", "oe_layernorm", "oe_moe_dense_relu2", "oe_tanh_rows", "oe_rot_norm_kv_write", "oe_token_shift_mix", "oe_last_rows_to_state",
           "oe_rope_split_kv_write", "oe_attn_split", "oe_moe_dense_act", "oe_group_rmsnorm", "oe_poly_norm",
           "oe_side_gate", "oe_latent_write", "oe_attn_latent", "oe_head_matmul", "oe_dyt_norm", "oe_pair_embed",
-          "oe_qkv_norm_rot_write", "oe_unrotate_heads"}
+          "oe_qkv_norm_rot_write", "oe_unrotate_heads", "oe_qkv_row_norm_rot_write", "oe_causal_conv", "oe_conv_rows_state",
+          "oe_selective_scan", "oe_selective_step"}
 _fn_cache: dict[str, object] = {}
 
 
@@ -195,8 +206,9 @@ def _i32(t: torch.Tensor, name: str) -> None:
 
 # ----------------------------------------------------------------------------------------
 
-def embed_gather(x: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, err: torch.Tensor | None) -> None:
-    """x[t] = table[ids[t]] as float32; ids outside the table set err[0] = 1 and give zeros."""
+def embed_gather(x: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, err: torch.Tensor | None,
+                 scale: float = 1.0) -> None:
+    """x[t] = table[ids[t]] * scale as float32; ids outside the table set err[0] = 1 and give zeros."""
     _dev(x, table, ids, err)
     _i32(ids, "ids")
     n, D = x.shape
@@ -205,7 +217,7 @@ def embed_gather(x: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, err: t
     if ids.numel() < n:
         raise KernelError("embed_gather: fewer ids than rows")
     _check(_fn("elementwise", "oe_embed_gather", table.dtype)(
-        _ptr(x), _ptr(table), _ptr(ids), n, D, table.shape[0], _ptr(err), _stream()), "embed_gather")
+        _ptr(x), _ptr(table), _ptr(ids), n, D, table.shape[0], float(scale), _ptr(err), _stream()), "embed_gather")
 
 
 def rmsnorm(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, eps: float) -> None:
@@ -361,6 +373,27 @@ def rmsnorm_add(dst: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float,
                                             int(bool(accumulate)), _ptr(cast_out), _stream()), "rmsnorm_add")
 
 
+def rmsnorm_sum(x: torch.Tensor, parts, w: torch.Tensor, alpha: float, eps: float, coef: float = 1.0,
+                cast_out: torch.Tensor | None = None) -> None:
+    """x = R(alpha x + s) * w with R(v) = v / sqrt(mean(v^2) + eps), all float32.  parts [(y, None)]: s = y; parts
+    [(y0, w0), (y1, w1)]: s = coef * (R(y0) * w0 + R(y1) * w1).  cast_out: a contiguous bfloat16 tensor of x's shape that
+    receives the new x, rounded."""
+    (y0, w0), (y1, w1) = parts[0], parts[1] if len(parts) > 1 else (None, None)
+    if len(parts) > 2 or (w0 is None) != (len(parts) == 1) or (w1 is None) != (len(parts) == 1):
+        raise KernelError("rmsnorm_sum: one output without a weight, or two with weights")
+    _dev(x, y0, w0, y1, w1, w, cast_out)
+    rows, D = x.shape
+    for t, n in ((x, "x"), (y0, "y0"), (y1, "y1"), (w0, "w0"), (w1, "w1"), (w, "w")):
+        if t is not None:
+            _f32c(t, n)
+            if t.numel() != (D if n[0] == "w" else rows * D):
+                raise KernelError(f"rmsnorm_sum: {n} does not have the stream's size")
+    if cast_out is not None and (cast_out.dtype != torch.bfloat16 or cast_out.shape != x.shape or not cast_out.is_contiguous()):
+        raise KernelError("rmsnorm_sum: cast_out must be contiguous bfloat16 of x's shape")
+    _check(_fn("rowwise", "oe_rmsnorm_sum")(_ptr(x), _ptr(y0), _ptr(w0), _ptr(y1), _ptr(w1), float(coef), float(alpha), _ptr(w),
+                                            rows, D, float(eps), _ptr(cast_out), _stream()), "rmsnorm_sum")
+
+
 def relu2_(a: torch.Tensor) -> None:
     """a = max(a, 0)^2 in place."""
     _dev(a)
@@ -499,13 +532,29 @@ def _unrotate_tables(unrotate, dv: int, what: str):
     return uc, us
 
 
+GATE_VALUE, GATE_HEAD = 1, 2     # must equal OE_GATE_* of common.cuh
+
+
+def _gate_args(gate, out: torch.Tensor, n_heads: int, dv: int, what: str) -> tuple:
+    """(pointer, row stride, mode) of an output gate: [T, H dv] or [T, H] of out's type, rows contiguous, or None."""
+    if gate is None:
+        return None, 0, 0
+    _dev(gate)
+    if gate.dtype != out.dtype or gate.dim() != 2 or gate.shape[0] < out.shape[0] or gate.stride(1) != 1 \
+            or gate.shape[1] not in (n_heads * dv, n_heads):
+        raise KernelError(f"{what}: the gate must be rows of H dv or H values of out's type")
+    return gate.data_ptr(), gate.stride(0), GATE_VALUE if gate.shape[1] == n_heads * dv else GATE_HEAD
+
+
 def attn_split(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, tables: torch.Tensor,
                tok_seq: torch.Tensor, tok_pos: torch.Tensor, n_heads: int, n_kv_heads: int, dk: int, dv: int,
-               window: int, scale: float, cap: float = 0.0, sinks: torch.Tensor | None = None, unrotate=None) -> None:
+               window: int, scale: float, cap: float = 0.0, sinks: torch.Tensor | None = None, unrotate=None,
+               gate: torch.Tensor | None = None) -> None:
     """out[t] = softmax attention of token t's query heads over the keys (pos - window, pos] of its sequence, with
     s <- cap tanh(s / cap) when cap > 0.  q [T, >= H dk] (row stride free), out contiguous [T, H dv].  sinks (float32
     [H] or None): exp(sinks[h]) is one more term of head h's denominator, without key or value.  unrotate ((cos, sin)
-    float32 [positions, dv/2] or None): every head's result is turned back by its query's position before it is stored."""
+    float32 [positions, dv/2] or None): every head's result is turned back by its query's position before it is stored.
+    gate ([T, H dv] or [T, H] of out's type, or None): the result is multiplied by the gate's sigmoid where it is stored."""
     _dev(out, q, kcache, vcache, tables, tok_seq, tok_pos, sinks)
     uc, us = _unrotate_tables(unrotate, dv, "attn_split")
     if sinks is not None:
@@ -522,7 +571,7 @@ def attn_split(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache:
     _check(_fn("attention_split", "oe_attn_split", out.dtype)(
         _ptr(out), _ptr(q), q.stride(0), _ptr(kcache), _ptr(vcache), _ptr(tables), tables.shape[1], _ptr(tok_seq),
         _ptr(tok_pos), out.shape[0], n_heads, n_kv_heads, dk, dv, int(window), float(scale), float(cap or 0.0),
-        _ptr(sinks), _ptr(uc), _ptr(us), _stream()), "attn_split")
+        _ptr(sinks), _ptr(uc), _ptr(us), *_gate_args(gate, out, n_heads, dv, "attn_split"), _stream()), "attn_split")
 
 
 # ---------------------------------------------------------------------------------------- attention_prep.cu
@@ -574,6 +623,42 @@ def qkv_norm_rot_write(q_out: torch.Tensor, kcache: torch.Tensor, vcache: torch.
         _ptr(kw), float(eps), _ptr(ck), _ptr(sk), int(rot_dims if ck is not None else 0), _ptr(cv), _ptr(sv),
         int(bool(value_norm)), _ptr(tables), tables.shape[1], _ptr(tok_seq), _ptr(tok_pos), T, n_heads, n_kv_heads, dk, dv,
         _stream()), "qkv_norm_rot_write")
+
+
+def qkv_row_norm_rot_write(qkv: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, norm_weights, eps: float,
+                           key_tables, rot_dims: int, pairing: str, tables: torch.Tensor, tok_seq: torch.Tensor,
+                           tok_pos: torch.Tensor, n_heads: int, n_kv_heads: int, dk: int, dv: int) -> None:
+    """From rows qkv [T, >= H dk + G dk + G dv] = [q | k | v]: q is divided by the root mean square of ALL its H dk values
+    (eps inside the root) and multiplied by norm_weights[0] (float32 [H dk]), k likewise over its G dk values
+    (norm_weights None: no norm); then the first rot_dims dimensions of every head are turned by the position (key_tables =
+    (cos, sin) float32 [positions, rot_dims/2] or None), 2i paired with 2i + 1 (pairing "interleaved") or i with
+    i + rot_dims/2 ("halves").  q is written back in place, k and v to the token's rows of the cache."""
+    qw, kw = norm_weights if norm_weights is not None else (None, None)
+    cos, sin = key_tables if key_tables is not None and rot_dims else (None, None)
+    _dev(qkv, kcache, vcache, qw, kw, cos, sin, tables, tok_seq, tok_pos)
+    for t, n in ((tables, "tables"), (tok_seq, "tok_seq"), (tok_pos, "tok_pos")):
+        _i32(t, n)
+    T = qkv.shape[0]
+    if qkv.dtype not in _SUFFIX or qkv.stride(1) != 1 or qkv.shape[1] < n_heads * dk + n_kv_heads * (dk + dv):
+        raise KernelError("qkv_row_norm_rot_write: qkv must be rows of at least H dk + G (dk + dv) values")
+    if not _split_cache_ok(kcache, vcache, qkv.dtype, n_kv_heads, dk, dv):
+        raise KernelError("qkv_row_norm_rot_write: the cache must be [pages, G, PAGE, dk] and [pages, G, PAGE, dv] of qkv's dtype")
+    for t, n, size in ((qw, "q norm weight", n_heads * dk), (kw, "k norm weight", n_kv_heads * dk)):
+        if t is not None:
+            _f32c(t, n)
+            if t.numel() != size:
+                raise KernelError(f"qkv_row_norm_rot_write: {n} must hold {size} values")
+    if (qw is None) != (kw is None):
+        raise KernelError("qkv_row_norm_rot_write: q and k are normed together or not at all")
+    if cos is not None:
+        _f32c(cos, "cos")
+        _f32c(sin, "sin")
+        if rot_dims % 2 or rot_dims > dk or cos.shape[1] != rot_dims // 2 or sin.shape != cos.shape:
+            raise KernelError("qkv_row_norm_rot_write: tables must be [positions, rot_dims/2], rot_dims even and <= dk")
+    _check(_fn("attention_prep", "oe_qkv_row_norm_rot_write", qkv.dtype)(
+        _ptr(qkv), qkv.stride(0), _ptr(kcache), _ptr(vcache), _ptr(qw), _ptr(kw), float(eps), _ptr(cos), _ptr(sin),
+        int(rot_dims if cos is not None else 0), {"interleaved": 0, "halves": 1}[pairing], _ptr(tables), tables.shape[1],
+        _ptr(tok_seq), _ptr(tok_pos), T, n_heads, n_kv_heads, dk, dv, _stream()), "qkv_row_norm_rot_write")
 
 
 def unrotate_heads(o: torch.Tensor, value_tables, tok_seq: torch.Tensor, tok_pos: torch.Tensor, n_heads: int,
@@ -722,6 +807,103 @@ def gdelta_scan(o: torch.Tensor, state: torch.Tensor, packed: torch.Tensor, v: t
         dv, _stream()), "gdelta_scan")
 
 
+# ---------------------------------------------------------------------------------------- selective_scan.cu
+
+def causal_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, state: torch.Tensor,
+                ctx) -> None:
+    """out[t, c] = silu(sum_j w[c, j] x[t - (taps - 1) + j, c] + bias[c]) over each sequence's rows, the rows before the
+    step's first from state [slots, max(taps - 1, 1), C] (float32), which then receives the sequence's last taps - 1 rows.
+    out [T, C] contiguous and x [T, >= C] (row stride free) of one dtype; w float32 [C, taps], bias float32 [C] or None."""
+    _dev(out, x, w, bias, state)
+    T, C = out.shape
+    taps = w.shape[1]
+    for t, n in ((w, "w"), (state, "state")) + (((bias, "bias"),) if bias is not None else ()):
+        _f32c(t, n)
+    if x.dtype != out.dtype or out.dtype not in _SUFFIX or not out.is_contiguous() or x.stride(1) != 1 or x.shape[0] < T \
+            or x.shape[1] < C or w.shape[0] != C or tuple(state.shape[1:]) != (max(taps - 1, 1), C) \
+            or (bias is not None and bias.numel() != C):
+        raise KernelError("causal_conv: shapes do not agree")
+    one_each = bool(ctx.all_decode and ctx.n_tokens == ctx.n_seqs) and 2 <= taps <= 4
+    _check(_fn("selective_scan", "oe_causal_conv", out.dtype)(
+        _ptr(out), _ptr(x), x.stride(0), _ptr(w), _ptr(bias), taps, _ptr(state), _ptr(ctx.tok_seq), _ptr(ctx.seq_slot),
+        _ptr(ctx.cu_q), T, ctx.n_seqs, C, int(one_each), _stream()), "causal_conv")
+    if taps > 1 and not one_each:
+        _check(_fn("selective_scan", "oe_conv_rows_state", out.dtype)(
+            _ptr(state), _ptr(x), x.stride(0), C, taps, _ptr(ctx.seq_slot), _ptr(ctx.cu_q), ctx.n_seqs, _stream()),
+            "conv_rows_state")
+
+
+def thin_cast(out: torch.Tensor, x: torch.Tensor) -> None:
+    """out (bfloat16 [T, n], contiguous) = the first n columns of x (float32 [T, >= n], row stride free)."""
+    _dev(out, x)
+    if out.dtype != torch.bfloat16 or not out.is_contiguous() or x.dtype != torch.float32 or x.stride(1) != 1 \
+            or x.shape[0] < out.shape[0] or x.shape[1] < out.shape[1]:
+        raise KernelError("thin_cast: out contiguous bfloat16, x float32 rows of at least as many values")
+    _check(_fn("selective_scan", "oe_thin_cast")(_ptr(out), _ptr(x), x.stride(0), out.shape[0], out.shape[1], _stream()),
+           "thin_cast")
+
+
+def _scan_shapes(what, y, state, u, dt_bias, thin, off_b, off_c, A2, Dw, z) -> tuple:
+    T, C = y.shape
+    N = A2.shape[1]
+    _dev(y, state, u, dt_bias, thin, A2, Dw, z)
+    for t, n in ((state, "state"), (dt_bias, "dt_bias"), (A2, "A2"), (Dw, "D")):
+        _f32c(t, n)
+    if y.dtype not in _SUFFIX or u.dtype != y.dtype or z.dtype != y.dtype or not (y.is_contiguous() and u.is_contiguous()) \
+            or tuple(u.shape) != (T, C) or z.stride(1) != 1 or z.shape[0] < T or z.shape[1] < C or A2.shape[0] != C \
+            or tuple(state.shape[1:]) != (C, N) or dt_bias.numel() != C or Dw.numel() != C or thin.dtype != torch.float32 \
+            or thin.stride(1) != 1 or thin.shape[0] < T or min(off_b, off_c) < 0 or max(off_b, off_c) + N > thin.shape[1]:
+        raise KernelError(f"{what}: shapes do not agree")
+    return T, C, N
+
+
+def selective_scan(y: torch.Tensor, state: torch.Tensor, u: torch.Tensor, zdt: torch.Tensor, dt_bias: torch.Tensor,
+                   thin: torch.Tensor, off_b: int, off_c: int, A2: torch.Tensor, Dw: torch.Tensor, z: torch.Tensor, ctx,
+                   segments=None) -> None:
+    """Per sequence and channel c, over the step's tokens in order: dt = softplus(zdt[c] + dt_bias[c]);
+    S[c, n] <- 2^(dt A2[c, n]) S[c, n] + dt u[c] b[n];  y[c] = (sum_n S[c, n] c[n] + Dw[c] u[c]) * silu(z[c]).
+    y, u [T, C] and z [T, >= C] of one dtype; zdt float32 [T, C]; thin float32 rows with b at column off_b, c at off_c;
+    state float32 [slots, C, N].  segments (seg_len, n_seg, seg_state, seg_dt; bfloat16 only): every sequence's tokens (at
+    most seg_len * n_seg) run as segments side by side, with float32 scratch [n_seqs, n_seg, C, N] and [n_seqs, n_seg, C];
+    the result differs from the one walk by the order of the sums only."""
+    T, C, N = _scan_shapes("selective_scan", y, state, u, dt_bias, thin, off_b, off_c, A2, Dw, z)
+    _dev(zdt)
+    _f32c(zdt, "zdt")
+    if tuple(zdt.shape) != (T, C):
+        raise KernelError("selective_scan: zdt must be [T, C]")
+    args = (_ptr(y), _ptr(state), _ptr(u), _ptr(zdt), _ptr(dt_bias), _ptr(thin), thin.stride(0), int(off_b), int(off_c), _ptr(A2),
+            _ptr(Dw), _ptr(z), z.stride(0), _ptr(ctx.seq_slot), _ptr(ctx.cu_q), ctx.n_seqs, C, N)
+    if segments is None:
+        _check(_fn("selective_scan", "oe_selective_scan", y.dtype)(*args, _stream()), "selective_scan")
+        return
+    seg_len, n_seg, seg_state, seg_dt = segments
+    _dev(seg_state, seg_dt)
+    _f32c(seg_state, "seg_state")
+    _f32c(seg_dt, "seg_dt")
+    if y.dtype != torch.bfloat16 or seg_len < 1 or n_seg < 1 or seg_len * n_seg < int(ctx.max_qlen) \
+            or seg_state.numel() < ctx.n_seqs * n_seg * C * N or seg_dt.numel() < ctx.n_seqs * n_seg * C:
+        raise KernelError("selective_scan: the segments do not cover the step's longest sequence, or their scratch is too small")
+    _check(_fn("selective_scan", "oe_selective_scan_segments")(*args, int(seg_len), int(n_seg), _ptr(seg_state), _ptr(seg_dt),
+                                                               _stream()), "selective_scan_segments")
+    LAUNCHES[0] += 2
+
+
+def selective_step(y: torch.Tensor, state: torch.Tensor, u: torch.Tensor, w_dt: torch.Tensor, off_r: int, rank: int,
+                   dt_bias: torch.Tensor, thin: torch.Tensor, off_b: int, off_c: int, A2: torch.Tensor, Dw: torch.Tensor,
+                   z: torch.Tensor, ctx) -> None:
+    """selective_scan for a step of one token per sequence, the product of the step sizes inside: zdt[c] = sum_j w_dt[c, j]
+    thin[off_r + j] over the rank.  w_dt [C, ldw] of y's dtype, ldw a multiple of 8, zeros behind the rank."""
+    T, C, N = _scan_shapes("selective_step", y, state, u, dt_bias, thin, off_b, off_c, A2, Dw, z)
+    _dev(w_dt)
+    if w_dt.dtype != y.dtype or not w_dt.is_contiguous() or w_dt.shape[0] != C or w_dt.shape[1] % 8 or not 1 <= rank <= w_dt.shape[1] \
+            or off_r < 0 or off_r + rank > thin.shape[1] or not (ctx.all_decode and ctx.n_tokens == ctx.n_seqs == T):
+        raise KernelError("selective_step: one token per sequence, w_dt [C, multiple of 8] of y's dtype")
+    _check(_fn("selective_scan", "oe_selective_step", y.dtype)(
+        _ptr(y), _ptr(state), _ptr(u), _ptr(w_dt), w_dt.shape[1], int(off_r), int(rank), _ptr(dt_bias), _ptr(thin),
+        thin.stride(0), int(off_b), int(off_c), _ptr(A2), _ptr(Dw), _ptr(z), z.stride(0), _ptr(ctx.seq_slot), _ptr(ctx.cu_q),
+        ctx.n_seqs, C, N, _stream()), "selective_step")
+
+
 # ---------------------------------------------------------------------------------------- retention.cu
 
 def retention_scan(o: torch.Tensor, state: torch.Tensor, proj: torch.Tensor, off_q: int, off_k: int, off_v: int,
@@ -781,8 +963,8 @@ def _route_arguments(n_experts: int, top: int, has_gate, weights: str, bias, gro
     """(gate, number of groups, groups that stay), checked."""
     if bias is not None:
         _f32c(bias, "bias")
-        if weights != "sigmoid" or bias.numel() != n_experts:
-            raise KernelError("moe_route: a choice bias needs sigmoid weights and one value per expert")
+        if bias.numel() != n_experts:
+            raise KernelError("moe_route: a bias needs one value per expert")
     if weights not in _ROUTE_MODES:
         raise KernelError(f"moe_route: weights must be one of {', '.join(_ROUTE_MODES)}, got {weights!r}")
     if top > n_experts:
@@ -800,8 +982,8 @@ def moe_route(z: torch.Tensor, n_experts: int, top: int, has_gate, dense: torch.
     (zero elsewhere) and, with has_gate, sigmoid of column E in its last column (has_gate "one": the constant 1, a
     shared expert without a gate; z needs no column for it); idx int32 [T, top] and wt float32 [T, top] receive the
     choice itself when given.  weights "softmax": the softmax over the `top` largest logits alone; "sigmoid": each
-    chosen expert's own sigmoid(logit), not renormalised.  bias (float32 [E], with "sigmoid" only): the choice is by
-    sigmoid(logit) + bias, the weights stay the sigmoids.  weights "softmax_all": the softmax over all experts, the chosen
+    chosen expert's own sigmoid(logit), not renormalised.  bias (float32 [E]): with "sigmoid" the choice is by
+    sigmoid(logit) + bias and the weights stay the sigmoids; else it is added to the logits.  weights "softmax_all": the softmax over all experts, the chosen
     scores divided by their sum (+ 1e-20).  groups (count, keep): the experts stand in `count` equal runs, only experts of
     the `keep` runs with the best single expert can be chosen."""
     _dev(z, dense, tok_seq, idx, wt, bias)
@@ -993,44 +1175,62 @@ def gla_scan(o: torch.Tensor, state: torch.Tensor, proj: torch.Tensor, off_q: in
 
 def latent_write(d: torch.Tensor | None, w: torch.Tensor | None, eps: float, q: torch.Tensor, qfull: torch.Tensor,
                  freq: torch.Tensor | None, dims: int, cache: torch.Tensor | None, tables: torch.Tensor, ctx, heads: int,
-                 dk: int, r: int, rd: int, write_cache: bool) -> None:
+                 dk: int, r: int, rd: int, write_cache: bool, tables_cs=None, halves: bool = False) -> None:
     """Per token: the first r values of d's row, divided by their root mean square and times w, and the last rd
     values with their first `dims` turned in pairs (2i, 2i + 1) by position * freq[i], go to the token's cache row
     [r + rd] (only when write_cache); the last rd dimensions of each of q's heads [dk + rd] are turned the same way
-    and written to qfull[t, h, r:].  d float32; q, qfull and cache of one dtype."""
-    _dev(d, w, q, qfull, freq, cache, tables)
+    and written to qfull[t, h, r:].  d float32 or of q's dtype; q, qfull and cache of one dtype.  tables_cs ((cos, sin)
+    float32 [positions, dims/2] or None): the angles come from there instead of from freq; halves: i is paired with
+    i + dims/2 instead of 2i with 2i + 1."""
+    cos, sin = tables_cs if tables_cs is not None else (None, None)
+    _dev(d, w, q, qfull, freq, cos, sin, cache, tables)
     T = q.shape[0]
     R = r + rd
     if q.stride(1) != 1 or q.shape[1] < heads * (dk + rd) or tuple(qfull.shape) != (T, heads * R) \
             or not qfull.is_contiguous() or q.dtype != qfull.dtype:
         raise KernelError("latent_write: q [T, >= H (dk + rd)], qfull contiguous [T, H (r + rd)] of q's dtype")
     if write_cache:
-        if d is None or w is None or cache is None or d.dtype != torch.float32 or d.stride(1) != 1 or d.shape[1] < R \
+        if d is None or w is None or cache is None or d.dtype not in (torch.float32, q.dtype) or d.stride(1) != 1 or d.shape[1] < R \
                 or w.dtype != torch.float32 or w.numel() != r or cache.dtype != q.dtype or not cache.is_contiguous() \
                 or tuple(cache.shape[1:]) != (PAGE, R):
-            raise KernelError("latent_write: d float32 [T, >= r + rd], w float32 [r], cache [pages, PAGE, r + rd]")
-    if dims and (freq is None or freq.dtype != torch.float32 or freq.numel() < dims // 2):
+            raise KernelError("latent_write: d float32 (or of q's dtype) [T, >= r + rd], w float32 [r], cache [pages, PAGE, r + rd]")
+    if dims and cos is not None:
+        _f32c(cos, "cos")
+        _f32c(sin, "sin")
+        if cos.dim() != 2 or cos.shape[1] != dims // 2 or sin.shape != cos.shape:
+            raise KernelError("latent_write: cos and sin must be [positions, dims / 2]")
+    elif dims and (freq is None or freq.dtype != torch.float32 or freq.numel() < dims // 2):
         raise KernelError("latent_write: freq float32 [dims / 2]")
-    _check(_fn("attention_latent", "oe_latent_write", q.dtype)(
+    _check(_fn("attention_latent", "oe_latent_write", q.dtype, in_dtype=torch.float32 if d is None else d.dtype)(
         _ptr(d), 0 if d is None else d.stride(0), _ptr(w), float(eps), _ptr(q), q.stride(0), _ptr(qfull), _ptr(freq),
-        int(dims), _ptr(cache), _ptr(tables), tables.shape[1], _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), T, heads, dk, r, rd,
+        _ptr(cos), _ptr(sin), int(dims), int(bool(halves)), _ptr(cache), _ptr(tables), tables.shape[1], _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), T, heads, dk, r, rd,
         int(bool(write_cache)), _stream()), "latent_write")
 
 
 def attn_latent(out: torch.Tensor, qfull: torch.Tensor, cache: torch.Tensor, tables: torch.Tensor, ctx, heads: int, r: int,
-                rd: int, scale: float) -> None:
+                rd: int, scale: float, window: int = 0, sinks: torch.Tensor | None = None,
+                gate: torch.Tensor | None = None) -> None:
     """out[t, h] = sum_j p_j c_j over the keys j <= pos of the token's sequence, p = softmax(scale * qfull[t, h] . row_j)
-    with row_j the cache row [r + rd] and c_j its first r values; float32 scores and sums."""
-    _dev(out, qfull, cache, tables)
+    with row_j the cache row [r + rd] and c_j its first r values; float32 scores and sums.  window (0: every key; n > 0: the
+    last n; -n: the query's own chunk of n), sinks (float32 [H]: exp(sinks[h]) joins the denominator), gate ([T, H] of out's
+    type: head h's output is multiplied by the gate's sigmoid)."""
+    _dev(out, qfull, cache, tables, sinks)
+    if sinks is not None:
+        _f32c(sinks, "sinks")
+        if sinks.numel() != heads:
+            raise KernelError("attn_latent: sinks must hold one value per query head")
     T = qfull.shape[0]
     R = r + rd
     if tuple(qfull.shape) != (T, heads * R) or tuple(out.shape) != (T, heads * r) or out.dtype != qfull.dtype \
             or cache.dtype != qfull.dtype or tuple(cache.shape[1:]) != (PAGE, R) \
             or not (out.is_contiguous() and qfull.is_contiguous() and cache.is_contiguous()):
         raise KernelError("attn_latent: shapes do not agree")
+    gp, gs, mode = _gate_args(gate, out, heads, r, "attn_latent")
+    if mode == GATE_VALUE and r > 1:
+        raise KernelError("attn_latent: the gate holds one value per head")
     _check(_fn("attention_latent", "oe_attn_latent", out.dtype)(
         _ptr(out), _ptr(qfull), _ptr(cache), _ptr(tables), tables.shape[1], _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), T, heads, r,
-        rd, float(scale), _stream()), "attn_latent")
+        rd, float(scale), int(window), _ptr(sinks), gp, gs, _stream()), "attn_latent")
 
 
 def head_matmul(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor) -> None:

@@ -612,22 +612,26 @@ def _attn_split_lib(dk: int, dv: int, shared: bool = False):
         fn = lib.oe_attn_split_mma
         fn.argtypes = [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                        c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p, c_void_p, c_void_p,
-                       c_void_p, c_void_p]
+                       c_void_p, c_void_p, c_longlong, c_int, c_void_p]
         fn.restype = c_int
         _split_libs[(dk, dv, shared)] = fn
     return fn
 
 
 def attention_split(out, q, kcache, vcache, tables, ctx, n_heads: int, n_kv_heads: int, dk: int, dv: int, window: int,
-                    scale: float, cap: float, sinks=None, unrotate=None) -> None:
+                    scale: float, cap: float, sinks=None, unrotate=None, gate=None) -> None:
     """out[t] = attention of token t's query heads over the keys (pos - window, pos] of its sequence, scores capped
     by cap tanh(s / cap) when cap > 0; bfloat16, q rotated already (rows of q may be a view of the fused product),
     kcache [pages, G, PAGE, dk], vcache [pages, G, PAGE, dv]; vcache None: the values are the first dv columns of the
     key rows.  sinks (float32 [H] or None): exp(sinks[h]) joins head h's denominator, without key or value.  unrotate
     ((cos, sin) float32 [positions, dv/2] or None): every head's result is turned back by its query's position, pair
     (m, m + dv/2), before it is stored (by the merge kernel when the keys are split).  window -n: the keys of the chunk of
-    n positions that the query lies in."""
+    n positions that the query lies in.  gate ([T, H dv] or [T, H] bfloat16, or None; the first kind not together with
+    unrotate): the result is multiplied by the gate's sigmoid where it is stored."""
     uc, us = ops._unrotate_tables(unrotate, dv, "attention_split")
+    gate_args = ops._gate_args(gate, out, n_heads, dv, "attention_split")
+    if gate_args[2] == ops.GATE_VALUE and (uc is not None or gate_args[0] % 4 or gate_args[1] % 2):
+        raise ops.KernelError("attention_split: a gate of one value per result needs 4-byte aligned rows and no turn back")
     if sinks is not None and (sinks.dtype != torch.float32 or not sinks.is_contiguous() or sinks.numel() != n_heads):
         raise ops.KernelError("attention_split: sinks must be float32, one value per query head")
     from .ops import PAGE
@@ -658,7 +662,8 @@ def attention_split(out, q, kcache, vcache, tables, ctx, n_heads: int, n_kv_head
                                    ctx.seq_qlen.data_ptr(), ctx.n_seqs, int(ctx.max_qlen), n_heads, n_kv_heads, int(window),
                                    float(scale), float(cap or 0.0), n_splits,
                                    None if partial is None else partial.data_ptr(),
-                                   None if sinks is None else sinks.data_ptr(), ops._ptr(uc), ops._ptr(us), ops._stream())
+                                   None if sinks is None else sinks.data_ptr(), ops._ptr(uc), ops._ptr(us), *gate_args,
+                                   ops._stream())
     ops._check(code, "attention_split_mma")
     if n_splits > 1:
         ops.LAUNCHES[0] += 1
@@ -672,11 +677,13 @@ def attention_latent_supported(n_heads: int, r: int, rd: int) -> bool:
     return r % 16 == 0 and attention_split_supported(r + rd, r, n_heads, 1)
 
 
-def attention_latent(out, qfull, rows, tables, ctx, n_heads: int, r: int, rd: int, scale: float) -> None:
+def attention_latent(out, qfull, rows, tables, ctx, n_heads: int, r: int, rd: int, scale: float, window: int = 0,
+                     sinks=None, gate=None) -> None:
     """out[t, h, :r] = sum_j p_j rows[j, :r] with p = softmax_j<=t(scale * qfull[t, h] . rows[j]); qfull [T, H (r + rd)]
-    (the queries taken through the key projection, the turned part behind), rows [pages, PAGE, r + rd]."""
+    (the queries taken through the key projection, the turned part behind), rows [pages, PAGE, r + rd].  window, sinks and
+    gate as attention_split's."""
     attention_split(out, qfull, rows.view(rows.shape[0], 1, rows.shape[1], r + rd), None, tables, ctx, n_heads, 1,
-                    r + rd, r, 0, scale, 0.0)
+                    r + rd, r, window, scale, 0.0, sinks, gate=gate)
 
 
 def head_matmul_supported(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:

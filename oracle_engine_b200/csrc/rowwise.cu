@@ -3,6 +3,9 @@
 //   cast_rows          y = x rounded to the compute type (a sublayer that reads the residual stream itself)
 //   rmsnorm_add        dst (+)= coef * (y / sqrt(mean(y^2) + eps)) * w        (all float32), optionally with a
 //                      copy of the new dst rounded to bfloat16 (the next sublayer's input)
+//   rmsnorm_sum        x = (v / sqrt(mean(v^2) + eps)) * w with v = alpha x + y, or v = alpha x + coef * (the sum of two
+//                      outputs, each divided by its own root mean square and times its own weight)   (all float32),
+//                      optionally with a copy of the new x rounded to bfloat16
 //   relu2              a = max(a, 0)^2 in place
 //   gelu               a = a (1 + erf(a / sqrt 2)) / 2 in place
 //   tanh_rows          y = tanh(x), float32 in, compute type out
@@ -77,6 +80,108 @@ rmsnorm_add_kernel(float* dst, const float* y, const float* __restrict__ w, int 
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
         const float v = (accumulate ? dr[d] : 0.f) + coef * ((yr[d] * s) * w[d]);
         dr[d] = v;
+        if (cr) cr[d] = __float2bfloat16_rn(v);
+    }
+}
+
+// Sums of up to two values a thread brings, over the block, in the order of block_sum.
+__device__ __forceinline__ void block_sum2(float& a, float& b, float* red) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+    a = warp_sum(a);
+    b = warp_sum(b);
+    if (lane == 0) { red[warp] = a; red[32 + warp] = b; }
+    __syncthreads();
+    a = warp_sum(lane < nwarps ? red[lane] : 0.f);
+    b = warp_sum(lane < nwarps ? red[32 + lane] : 0.f);
+}
+
+// One block per row, in registers up to 4,096 columns.  w0 null: v = alpha x + y0 (y1 and w1 are not read).
+__global__ void __launch_bounds__(256)
+rmsnorm_sum_kernel(float* x, const float* y0, const float* __restrict__ w0, const float* y1, const float* __restrict__ w1,
+                   float coef, float alpha, const float* __restrict__ w, int D, float eps, bf16* cast_out) {
+    __shared__ float red[64], red2[32];
+    constexpr int KEEP = 4;
+    pdl_launch_dependents();
+    pdl_wait();
+    float* xr = x + (size_t)blockIdx.x * D;
+    const float* ar = y0 + (size_t)blockIdx.x * D;
+    const float* br = w0 ? y1 + (size_t)blockIdx.x * D : ar;
+    bf16* cr = cast_out ? cast_out + (size_t)blockIdx.x * D : nullptr;
+    const bool vec = (D % 4 == 0) && D <= KEEP * 4 * 256 &&
+                     !(((uintptr_t)x | (uintptr_t)y0 | (uintptr_t)y1 | (uintptr_t)w | (uintptr_t)w0 | (uintptr_t)w1) & 15) &&
+                     !((uintptr_t)cast_out & 7);
+    if (vec) {
+        const int n4 = D / 4;
+        float4 v[KEEP], a[KEEP], b[KEEP];
+        float sa = 0.f, sb = 0.f;
+#pragma unroll
+        for (int j = 0; j < KEEP; j++) {
+            const int i = threadIdx.x + j * 256;
+            v[j] = a[j] = b[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < n4) {
+                v[j] = reinterpret_cast<const float4*>(xr)[i];
+                a[j] = reinterpret_cast<const float4*>(ar)[i];
+                if (w0) b[j] = reinterpret_cast<const float4*>(br)[i];
+            }
+            sa += a[j].x * a[j].x + a[j].y * a[j].y + a[j].z * a[j].z + a[j].w * a[j].w;
+            sb += b[j].x * b[j].x + b[j].y * b[j].y + b[j].z * b[j].z + b[j].w * b[j].w;
+        }
+        float ss = 0.f;
+        if (w0) {
+            block_sum2(sa, sb, red);
+            const float na = 1.f / sqrtf(sa / (float)D + eps), nb = 1.f / sqrtf(sb / (float)D + eps);
+#pragma unroll
+            for (int j = 0; j < KEEP; j++) {
+                const int i = threadIdx.x + j * 256;
+                if (i >= n4) continue;
+                const float4 p = reinterpret_cast<const float4*>(w0)[i], q = reinterpret_cast<const float4*>(w1)[i];
+                a[j].x = coef * (a[j].x * na * p.x + b[j].x * nb * q.x); a[j].y = coef * (a[j].y * na * p.y + b[j].y * nb * q.y);
+                a[j].z = coef * (a[j].z * na * p.z + b[j].z * nb * q.z); a[j].w = coef * (a[j].w * na * p.w + b[j].w * nb * q.w);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < KEEP; j++) {
+            v[j].x = fmaf(alpha, v[j].x, a[j].x); v[j].y = fmaf(alpha, v[j].y, a[j].y);
+            v[j].z = fmaf(alpha, v[j].z, a[j].z); v[j].w = fmaf(alpha, v[j].w, a[j].w);
+            ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+        }
+        ss = block_sum(ss, red2);
+        const float s = 1.f / sqrtf(ss / (float)D + eps);
+#pragma unroll
+        for (int j = 0; j < KEEP; j++) {
+            const int i = threadIdx.x + j * 256;
+            if (i >= n4) continue;
+            const float4 g = reinterpret_cast<const float4*>(w)[i];
+            const float4 d = make_float4(v[j].x * s * g.x, v[j].y * s * g.y, v[j].z * s * g.z, v[j].w * s * g.w);
+            reinterpret_cast<float4*>(xr)[i] = d;
+            if (cr) {
+                __nv_bfloat162 h[2] = {__floats2bfloat162_rn(d.x, d.y), __floats2bfloat162_rn(d.z, d.w)};
+                reinterpret_cast<uint2*>(cr)[i] = *reinterpret_cast<uint2*>(h);
+            }
+        }
+        return;
+    }
+    // any width: v goes through x itself; a thread reads back only what it wrote
+    float na = 1.f, nb = 1.f;
+    if (w0) {
+        float sa = 0.f, sb = 0.f;
+        for (int d = threadIdx.x; d < D; d += blockDim.x) { sa = fmaf(ar[d], ar[d], sa); sb = fmaf(br[d], br[d], sb); }
+        block_sum2(sa, sb, red);
+        na = 1.f / sqrtf(sa / (float)D + eps);
+        nb = 1.f / sqrtf(sb / (float)D + eps);
+    }
+    float ss = 0.f;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+        const float add = w0 ? coef * (ar[d] * na * w0[d] + br[d] * nb * w1[d]) : ar[d];
+        const float v = fmaf(alpha, xr[d], add);
+        xr[d] = v;
+        ss = fmaf(v, v, ss);
+    }
+    ss = block_sum(ss, red2);
+    const float s = 1.f / sqrtf(ss / (float)D + eps);
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+        const float v = xr[d] * s * w[d];
+        xr[d] = v;
         if (cr) cr[d] = __float2bfloat16_rn(v);
     }
 }
@@ -278,6 +383,13 @@ int oe_rmsnorm_add(float* dst, const float* y, const float* w, int rows, int D, 
                    bf16* cast_out, cudaStream_t st) {
     if (rows <= 0) return 0;
     return oe_launch(rmsnorm_add_kernel, dim3(rows), dim3(256), 0, st, dst, y, w, D, eps, coef, accumulate, cast_out);
+}
+
+int oe_rmsnorm_sum(float* x, const float* y0, const float* w0, const float* y1, const float* w1, float coef, float alpha,
+                   const float* w, int rows, int D, float eps, bf16* cast_out, cudaStream_t st) {
+    if (rows <= 0) return 0;
+    if (D < 1 || (w0 != nullptr && (y1 == nullptr || w1 == nullptr))) return OE_ERR_UNSUPPORTED;
+    return oe_launch(rmsnorm_sum_kernel, dim3(rows), dim3(256), 0, st, x, y0, w0, y1, w1, coef, alpha, w, D, eps, cast_out);
 }
 
 int oe_relu2_f32(float* a, long long total, cudaStream_t st) {

@@ -60,26 +60,28 @@ def split_mixer_core(rt, out, qkv, cos, sin, rot, kcache, vcache, tables, ctx, H
 
 
 def split_attend(rt, out, q, kcache, vcache, tables, ctx, H, G, dk, dv, window, scale, cap, sinks=None,
-                 unrotate=None) -> None:
+                 unrotate=None, gate=None) -> None:
     """Attention of queries that are turned already over keys and values that lie in two cache tensors; `sinks`
     (float32 [H] or None): a learned score per head that joins the softmax's denominator without key or value;
     `unrotate` ((cos, sin) tables [positions, dv/2] or None): every head's result is turned back by its query's
-    position inside the kernel that stores it."""
+    position inside the kernel that stores it; `gate` (of out's type, [T, H dv] one value per result or [T, H] one per
+    head, or None): the result is multiplied by sigmoid(gate) where it is stored."""
     if rt.dtype == torch.bfloat16 and rt.tensor_cores:
         from ..csrc import ops_tc
         if ops_tc.attention_split_supported(dk, dv, H, G):
-            ops_tc.attention_split(out, q, kcache, vcache, tables, ctx, H, G, dk, dv, window, scale, cap, sinks, unrotate)
+            ops_tc.attention_split(out, q, kcache, vcache, tables, ctx, H, G, dk, dv, window, scale, cap, sinks, unrotate,
+                                   gate)
             return
     ops.attn_split(out, q, kcache, vcache, tables, ctx.tok_seq, ctx.tok_pos, H, G, dk, dv, window, scale, cap, sinks,
-                   unrotate)
+                   unrotate, gate)
 
 
-def latent_core(rt, out, qfull, rows, tables, ctx, H, r, rd, scale) -> None:
+def latent_core(rt, out, qfull, rows, tables, ctx, H, r, rd, scale, window=0, sinks=None, gate=None) -> None:
     """Attention of absorbed queries [T, H (r + rd)] over a cache of latent rows [r + rd]; out [T, H r] gets each
-    head's weighted sum of the latents (parts/latent_attention.py)."""
+    head's weighted sum of the latents (parts/latent_attention.py).  window, sinks, gate ([T, H]): as split_attend's."""
     if rt.dtype == torch.bfloat16 and rt.tensor_cores:
         from ..csrc import ops_tc
         if ops_tc.attention_latent_supported(H, r, rd):
-            ops_tc.attention_latent(out, qfull, rows, tables, ctx, H, r, rd, scale)
+            ops_tc.attention_latent(out, qfull, rows, tables, ctx, H, r, rd, scale, window, sinks, gate)
             return
-    ops.attn_latent(out, qfull, rows, tables, ctx, H, r, rd, scale)
+    ops.attn_latent(out, qfull, rows, tables, ctx, H, r, rd, scale, window, sinks, gate)

@@ -3,6 +3,8 @@ the reference's layer (core/model.cpp:361-474).  The mixer and the feed-forward 
 outputs into the float32 residual stream themselves (fused into their last product).
 `norm_after`: x += norm(mixer(x)); x += norm(ffn(x)): the sublayers read the residual stream itself and
 their OUTPUT is normed before it is added; a sublayer adds its output into a zeroed float32 buffer.
+`norm_of_sum`: x <- norm(alpha x + mixer(x)); x <- norm(alpha x + ffn(x)): the norm takes the sum, so the stream is its
+output.
 `pre_norm_scaled`: x += m * s1 * mixer(norm(x)); x += m * s2 * ffn(norm(x)) with m one constant and s1, s2 one
 weight per channel each (a layer scale).
 `parallel_sublayers`: h = norm(x); x += mixer(h) + ffn(h): one norm, both sublayers read its output.
@@ -164,6 +166,50 @@ class NormAfterBlock:
                 y.zero_()
                 self.feed_forward.forward(h, y, ctx)
             self.ffn_norm.add_into(x, y, keep_cast=True)
+
+
+@BLOCKS.register("norm_of_sum")
+class NormOfSumBlock:
+    """x <- norm_1(alpha x + mixer(x)); x <- norm_2(alpha x + ffn(x)) (the second only with a feed-forward).
+    params: alpha (default 1).  A mixer made of mixers with output norms (`normed_outputs`) hands its outputs over as they
+    are, and one kernel norms them, adds them and norms the sum."""
+
+    def __init__(self, mixer, feed_forward, mixer_norm, ffn_norm, params, prefix, runtime):
+        if mixer_norm is None or (feed_forward is not None and ffn_norm is None):
+            raise ValueError("norm_of_sum: every sublayer needs the norm of its sum")
+        self.mixer, self.feed_forward, self.mixer_norm, self.ffn_norm = mixer, feed_forward, mixer_norm, ffn_norm
+        self.rt = runtime
+        self.alpha = float(params.get("alpha", 1.0))
+
+    def parts(self):
+        return [p for p in (self.mixer, self.mixer_norm, self.feed_forward, self.ffn_norm) if p is not None]
+
+    def first_weights(self):
+        return _first_weights(self.mixer)
+
+    def _output(self, part, h, x, *args):
+        """The sublayer's output in a float32 buffer of the stream's shape."""
+        y = self.rt.buffer("sublayer_out", *x.shape, dtype=torch.float32)
+        if getattr(part, "can_overwrite", False):
+            part.forward(h, y, *args, overwrite=True)
+        else:
+            y.zero_()
+            part.forward(h, y, *args)
+        return y
+
+    def forward(self, x, ctx, cache, state, owns_cache=True):
+        self.rt.next_weights = None
+        h = self.rt.activations(x)
+        outputs = getattr(self.mixer, "normed_outputs", None)
+        parts = None
+        if outputs is not None and getattr(self.mixer, "eps", None) == self.mixer_norm.eps:
+            parts = outputs(h, ctx, cache, state, owns_cache)
+        if parts is not None:
+            self.mixer_norm.sum_into(x, parts, self.alpha, coef=1.0 / len(parts))
+        else:
+            self.mixer_norm.sum_into(x, [(self._output(self.mixer, h, x, ctx, cache, state, owns_cache), None)], self.alpha)
+        if self.feed_forward is not None:
+            self.ffn_norm.sum_into(x, [(self._output(self.feed_forward, self.rt.activations(x), x, ctx), None)], self.alpha)
 
 
 class ChannelScales(Part):

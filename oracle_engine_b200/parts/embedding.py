@@ -1,7 +1,7 @@
 """Token embedding and output head.
 
-`token_embedding`: x = E[token] as float32 (core/model.cpp:352-358); an id outside the
-table is an error, not clamped.  `lm_head`: logits = W x in float32, W a separate matrix
+`token_embedding`: x = E[token] as float32 (core/model.cpp:352-358), optionally times a constant; an id outside
+the table is an error, not clamped.  `lm_head`: logits = W x in float32, W a separate matrix
 or, when tied, the embedding table (core/model.cpp:482-492); an optional constant `scale` multiplies the logits,
 an optional `softcap` c bounds them, c tanh(z / c).
 `pair_hash_embedding`: x = E[token] * scale + P[hash(previous token, token)], a second table indexed by a hash of
@@ -18,7 +18,7 @@ from .spec import StateNeed, TensorDecl
 
 @EMBEDDINGS.register("token_embedding")
 class TokenEmbedding(Part):
-    """params: vocab_size, hidden_size, name."""
+    """params: vocab_size, hidden_size, name, scale (a constant the row is multiplied by in float32; default 1)."""
     graph_safe = True
 
     def __init__(self, params, prefix, runtime):
@@ -26,6 +26,7 @@ class TokenEmbedding(Part):
         self.V = int(self._need("vocab_size"))
         self.D = int(self._need("hidden_size"))
         self.name = prefix + self._need("name")
+        self.scale = float(self.params.get("scale", 1.0))
         self.table = None
         self.err = None
 
@@ -39,7 +40,7 @@ class TokenEmbedding(Part):
     def forward(self, ids, n_tokens, out=None):
         """The residual stream [n_tokens, hidden] float32 (written into `out` if given)."""
         x = self.rt.empty(n_tokens, self.D, dtype=torch.float32) if out is None else out
-        ops.embed_gather(x, self.table, ids, self.err)
+        ops.embed_gather(x, self.table, ids, self.err, self.scale)
         return x
 
 

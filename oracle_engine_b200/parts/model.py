@@ -18,6 +18,7 @@ from . import delta_rule, parallel, sink_attention, time_mix  # noqa: F401,E402
 from . import capped_attention, moe, retention  # noqa: F401,E402
 from . import gla, latent_attention  # noqa: F401,E402
 from . import general_delta, passes, rotated_value_attention  # noqa: F401,E402
+from . import gated_attention, selective_scan  # noqa: F401,E402
 
 
 class DecoderModel:

@@ -6,7 +6,8 @@
 Variants by parameter: the weights may be each chosen expert's own sigmoid(z_e), not renormalised; the weight may
 multiply the expert's input, y = sum_chosen E_e(w_e h) (its gate and up rows are linear in the input, so the kernel
 scales those: silu(w_e g) * (w_e u)); the shared expert may be added without a gate; the choice may be by
-sigmoid(z_e) + a learned bias per expert while the weights stay the sigmoids; the experts' unit may be clamped and
+sigmoid(z_e) + a learned bias per expert while the weights stay the sigmoids; the logits may have a learned bias of
+their own, z = Wr h + br; the experts' unit may be clamped and
 shifted, g = min(Wgate h, L), u = clamp(Wup h, -L, L), E_e(h) = Wdown_e (g * sigmoid(1.702 g) * (u + 1)).
 
 Choice by groups (`groups`, a variant of both kinds): the experts stand in `count` equal runs, a run's score is its best
@@ -66,8 +67,8 @@ class MoESwiGLU(Part):
     sigmoid(logit), not renormalised), weight_on ("output", the default: y = sum w_e E_e(h); "input": y = sum E_e(w_e h)),
     shared_gate (default True: the shared expert's output times sigmoid(Wsg h); False: added as it is), choice_bias
     (True: a tensor of one value per expert is added to the sigmoids for the choice alone; needs router_weights
-    "sigmoid"), activation ("silu", the default, or "clamped" with `limit`), groups (None, or {"count", "keep"}), tensor_names (optional overrides of
-    "expert" (a format with {e}), "router", "shared", "shared_gate", "choice_bias")."""
+    "sigmoid"), router_bias (True: a tensor of one value per expert is part of the logits; not with "sigmoid"), activation ("silu", the default, or "clamped" with `limit`), groups (None, or {"count", "keep"}), tensor_names (optional overrides of
+    "expert" (a format with {e}), "router", "router_bias", "shared", "shared_gate", "choice_bias")."""
 
     def __init__(self, params, prefix, runtime):
         super().__init__(params, prefix, runtime)
@@ -83,6 +84,7 @@ class MoESwiGLU(Part):
         if self.router_weights not in ("softmax", "sigmoid", "softmax_all") or self.weight_on not in ("output", "input"):
             raise ValueError("moe_swiglu: router_weights is softmax, sigmoid or softmax_all, weight_on is output or input")
         self.choice_bias = bool(self.params.get("choice_bias", False))
+        self.router_bias = bool(self.params.get("router_bias", False))
         self.activation = self.params.get("activation") or "silu"
         self.limit = float(self.params.get("limit") or 0.0)
         if self.activation not in ("silu", "clamped") or (self.activation == "clamped" and not self.limit > 0):
@@ -91,12 +93,14 @@ class MoESwiGLU(Part):
             raise ValueError("moe_swiglu: the clamped unit is not linear in its input; its weight goes on the output")
         if self.choice_bias and self.router_weights != "sigmoid":
             raise ValueError("moe_swiglu: a choice bias is added to sigmoids; router_weights must be sigmoid")
+        if self.router_bias and self.router_weights == "sigmoid":
+            raise ValueError("moe_swiglu: a bias on the logits goes with weights that are a softmax")
         if not 1 <= self.top <= self.E:
             raise ValueError(f"moe_swiglu: top {self.top} of {self.E} experts")
         if self.E > 1024:
             raise ValueError("moe_swiglu: up to 1,024 experts are supported")
         names = {"expert": "mlp.e{e}.", "router": "mlp.router", "shared": "mlp.shared.", "shared_gate": "mlp.shared.sg",
-                 "choice_bias": "mlp.correction",
+                 "choice_bias": "mlp.correction", "router_bias": "mlp.router.b",
                  **self.params.get("tensor_names", {})}
         self.names = {k: prefix + v for k, v in names.items()}
         self.F = self.E * self.ff + self.sff
@@ -117,6 +121,8 @@ class MoESwiGLU(Part):
             out.append(TensorDecl(self.names["shared_gate"], (1, self.D)))
         if self.choice_bias:
             out.append(TensorDecl(self.names["choice_bias"], (self.E,)))
+        if self.router_bias:
+            out.append(TensorDecl(self.names["router_bias"], (self.E,)))
         return out
 
     def load(self, get):
@@ -128,6 +134,8 @@ class MoESwiGLU(Part):
         self.w_route = torch.cat(route, 0).contiguous()
         if self.choice_bias:
             self.bias = self.rt.to_f32(get(self.names["choice_bias"]))
+        if self.router_bias:
+            self.bias = self.rt.to_f32(get(self.names["router_bias"]))
 
     def weight_bytes(self):
         return sum(t.numel() * t.element_size() for t in (self.w_gu, self.w_down, self.w_route) if t is not None)

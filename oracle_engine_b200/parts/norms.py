@@ -2,7 +2,8 @@
 computed in float32 and stored in the compute dtype (reference: core/ops.cpp:149-195; the
 epsilon is a parameter here, always passed).  `add_into(dst, y, coef)` is the same norm applied to a
 sublayer's float32 OUTPUT and added, times coef, into another float32 tensor (layers that norm what
-a sublayer returns instead of what it reads).  With `groups` > 1 the row is cut into that many equal consecutive parts
+a sublayer returns instead of what it reads); `sum_into(x, parts, alpha)` norms the sum of alpha x and what a sublayer returned, in place (layers
+whose stream is itself a norm's output).  With `groups` > 1 the row is cut into that many equal consecutive parts
 and each part is divided by its own root mean square (the weight still spans the whole row).
 `dynamic_tanh`: y = tanh(alpha x) * w + b with one scalar alpha and the vectors w, b: a norm that computes no
 mean and no variance, so every value of a row is normed by itself.
@@ -53,16 +54,29 @@ class RMSNorm(Part):
     def add_into(self, dst, y, coef: float = 1.0, accumulate: bool = True, keep_cast: bool = False) -> None:
         """dst (+)= coef * norm(y); dst and y float32 of one shape.  keep_cast: on the bfloat16 path the kernel
         also leaves the new dst rounded to bfloat16 for the sublayer that reads it next (Runtime.activations)."""
-        cast = None
-        if keep_cast and self.rt.dtype != dst.dtype:
-            # two buffers in turn: the copy a sublayer is reading stays while the next one is written
-            self.rt._cast_turn ^= 1
-            cast = self.rt.buffer(f"stream_copy{self.rt._cast_turn}", *dst.shape)
-            self.rt.cast_cache = (dst.data_ptr(), cast)
+        cast = self._cast_buffer(dst) if keep_cast else None
         if self.groups > 1:
             ops.group_rmsnorm_add(dst, y, self.weight, self.eps, self.groups, coef, accumulate, cast)
         else:
             ops.rmsnorm_add(dst, y, self.weight, self.eps, coef, accumulate, cast)
+
+
+    def sum_into(self, x, parts, alpha: float, coef: float = 1.0) -> None:
+        """x <- norm(alpha x + s): s the output y of parts [(y, None)], or coef times the sum of two outputs normed with
+        weights of their own, parts [(y0, w0), (y1, w1)] (ops.rmsnorm_sum); all float32.  On the bfloat16 path the kernel
+        also leaves the new x rounded for the sublayer that reads it next (Runtime.activations)."""
+        if self.groups > 1:
+            raise ValueError("rms_norm: the norm of a sum is not built in groups")
+        ops.rmsnorm_sum(x, parts, self.weight, alpha, self.eps, coef, self._cast_buffer(x))
+
+    def _cast_buffer(self, dst):
+        if self.rt.dtype == dst.dtype:
+            return None
+        # two buffers in turn: the copy a sublayer is reading stays while the next one is written
+        self.rt._cast_turn ^= 1
+        cast = self.rt.buffer(f"stream_copy{self.rt._cast_turn}", *dst.shape)
+        self.rt.cast_cache = (dst.data_ptr(), cast)
+        return cast
 
 
 @NORMS.register("layer_norm")

@@ -10,12 +10,17 @@ params: hidden_size, eps, branches: a list of {"tag", "kind", "params", "prefix"
 registered kind and parameters of the mixer, the tensor-name prefix below the layer's, and the name of its output
 norm's weight or its coefficient).  At most one branch may keep a paged cache (it gets the entry's); every
 branch's per-sequence state is kept under "<tag>.<name>".
+
+Branches that offer it (`joint_weight`, the attribute that holds the first matrix, and a forward that takes `projected`)
+have their first products computed as one, [W1; W2; ...] h, where the tensor-core kernels serve the shapes: once all have
+loaded, the matrices move into one and stay views of it.
 """
 from __future__ import annotations
 
 import torch
 
 from ..csrc import ops
+from .linear import chain_flags, matmul_nt
 from .registry import MIXERS, Part
 from .spec import TensorDecl
 
@@ -49,6 +54,7 @@ class ParallelMixers(Part):
             raise ValueError("parallel_mixers: only one branch may keep a paged cache")
         self.graph_safe = all(getattr(m, "graph_safe", False) for _, m, _ in self.branches)
         self.out_w = {}
+        self.w_joined, self.columns = None, []
 
     def tensors(self):
         out = []
@@ -61,6 +67,31 @@ class ParallelMixers(Part):
             m.load(get)
             if norm_name:
                 self.out_w[tag] = self.rt.to_f32(get(norm_name))
+        self._join()
+
+    def _join(self):
+        self.w_joined, self.columns = None, []
+        mixers = [m for _, m, _ in self.branches]
+        if len(mixers) < 2 or self.rt.dtype != torch.bfloat16 or not self.rt.tensor_cores \
+                or not all(hasattr(m, "joint_weight") for m in mixers):
+            return
+        mats = [getattr(m, m.joint_weight) for m in mixers]
+        # rows of 16-byte pieces: what reads a branch's columns starts on such a boundary
+        if self.D % 8 or any(w.shape[0] % 8 for w in mats):
+            return
+        self.w_joined, row = torch.cat(mats, 0), 0
+        for m, w in zip(mixers, mats):
+            setattr(m, m.joint_weight, self.w_joined[row:row + w.shape[0]])
+            self.columns.append((row, row + w.shape[0]))
+            row += w.shape[0]
+
+    def _projected(self, h):
+        """Per branch, the keyword arguments that hand over its part of the joined product."""
+        if self.w_joined is None:
+            return [{} for _ in self.branches]
+        y = self.rt.buffer("parallel.joined", h.shape[0], self.w_joined.shape[0])
+        matmul_nt(self.rt, y, h, self.w_joined, early=chain_flags("mixer_in", h.shape[0]))
+        return [{"projected": y[:, lo:hi]} for lo, hi in self.columns]
 
     def cache_need(self):
         for _, m, _ in self.branches:
@@ -81,28 +112,42 @@ class ParallelMixers(Part):
         return sum(m.flops(start, count) for _, m, _ in self.branches)
 
     def first_weights(self):
+        if self.w_joined is not None:
+            return self.w_joined
         f = getattr(self.branches[0][1], "first_weights", None)
         return f() if f is not None else None
 
     can_overwrite = True
 
-    def _branch_into(self, i, y, h, ctx, cache, state, owns_cache):
+    def _branch_into(self, i, y, h, ctx, cache, state, owns_cache, projected):
         tag, m, _ = self.branches[i]
         own = {name[len(tag) + 1:]: t for name, t in state.items() if name.startswith(tag + ".")}
         if getattr(m, "can_overwrite", False):
-            m.forward(h, y, ctx, cache, own, owns_cache, overwrite=True)
+            m.forward(h, y, ctx, cache, own, owns_cache, overwrite=True, **projected)
         else:
             y.zero_()
-            m.forward(h, y, ctx, cache, own, owns_cache)
+            m.forward(h, y, ctx, cache, own, owns_cache, **projected)
+
+    def normed_outputs(self, h, ctx, cache, state, owns_cache=True):
+        """[(a branch's output [T, hidden] float32, its norm's weight)]: the caller norms each with `eps` and takes their
+        mean.  None where the branches are not two with output norms."""
+        if self.weighted or len(self.branches) != 2:
+            return None
+        out = []
+        for i, (projected, (tag, _, _)) in enumerate(zip(self._projected(h), self.branches)):
+            y = self.rt.buffer(f"parallel.branch_out{i}", h.shape[0], self.D, dtype=torch.float32)
+            self._branch_into(i, y, h, ctx, cache, state, owns_cache, projected)
+            out.append((y, self.out_w[tag]))
+        return out
 
     def _forward_weighted(self, h, residual, ctx, cache, state, owns_cache, overwrite, scale):
         mult, vec = scale if scale is not None else (1.0, None)
         if overwrite:
             residual.zero_()
         ys = []
-        for i in range(len(self.branches)):
+        for i, projected in enumerate(self._projected(h)):
             y = self.rt.buffer(f"parallel.branch_out{i}", h.shape[0], self.D, dtype=torch.float32)
-            self._branch_into(i, y, h, ctx, cache, state, owns_cache)
+            self._branch_into(i, y, h, ctx, cache, state, owns_cache, projected)
             ys.append(y)
         for i in range(0, len(ys), 2):               # two outputs a kernel
             two = i + 1 < len(ys)
@@ -119,11 +164,6 @@ class ParallelMixers(Part):
             raise ValueError("parallel_mixers: branches with output norms take no scale")
         coef = 1.0 / len(self.branches)
         y = self.rt.buffer("parallel.branch_out", h.shape[0], self.D, dtype=torch.float32)
-        for i, (tag, m, _) in enumerate(self.branches):
-            own = {name[len(tag) + 1:]: t for name, t in state.items() if name.startswith(tag + ".")}
-            if getattr(m, "can_overwrite", False):
-                m.forward(h, y, ctx, cache, own, owns_cache, overwrite=True)
-            else:
-                y.zero_()
-                m.forward(h, y, ctx, cache, own, owns_cache)
+        for i, (projected, (tag, _, _)) in enumerate(zip(self._projected(h), self.branches)):
+            self._branch_into(i, y, h, ctx, cache, state, owns_cache, projected)
             ops.rmsnorm_add(residual, y, self.out_w[tag], self.eps, coef, accumulate=not (overwrite and i == 0))

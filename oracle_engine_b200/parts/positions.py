@@ -1,4 +1,4 @@
-"""Position encodings.  `rotary`: rotate-half RoPE with optional llama3 frequency scaling.
+"""Position encodings.  `rotary`: rotate-half RoPE with optional llama3 or YaRN frequency scaling.
 
 The reference computes theta_i = pos / base^(2i/hd) and its cosine and sine per token
 (core/ops.cpp:461-466) and has no frequency scaling.  Here the inverse frequencies are
@@ -9,6 +9,10 @@ llama3 scaling, with f_i = base^(-2i/hd) and wavelength l_i = 2 pi / f_i:
   l_i < orig/high_freq_factor          keep f_i
   l_i > orig/low_freq_factor           f_i / factor
   otherwise  s = (orig/l_i - low)/(high - low);  f_i' = (1-s) f_i/factor + s f_i
+
+YaRN scaling (`kind` "yarn"), with c(t) = dims ln(orig / (2 pi t)) / (2 ln base), the pair that makes t turns over orig
+positions:  lo = max(floor c(fast), 0), hi = min(ceil c(slow), dims - 1), r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1),
+f_i' = r_i f_i / factor + (1 - r_i) f_i, and cosine and sine are multiplied by 0.1 ln(factor) + 1.
 """
 from __future__ import annotations
 
@@ -25,6 +29,9 @@ def rotary_inv_freq(head_dim: int, theta: float, scaling: dict | None) -> torch.
     if not scaling:
         return f
     factor = float(scaling["factor"])
+    if scaling.get("kind") == "yarn":
+        r = _yarn_ramp(head_dim, theta, scaling)
+        return f / factor * r + f * (1.0 - r)
     low = float(scaling["low_freq_factor"])
     high = float(scaling["high_freq_factor"])
     orig = float(scaling["original_max_position_embeddings"])
@@ -42,9 +49,26 @@ def rotary_inv_freq(head_dim: int, theta: float, scaling: dict | None) -> torch.
     return out
 
 
+def _yarn_ramp(dims: int, theta: float, scaling: dict) -> torch.Tensor:
+    orig = float(scaling["original"])
+
+    def pair(turns):
+        return dims * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+    lo = max(math.floor(pair(float(scaling["fast"]))), 0)
+    hi = min(math.ceil(pair(float(scaling["slow"]))), dims - 1)
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    return ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+
+
+def rotary_magnitude(scaling: dict | None) -> float:
+    """What cosine and sine are multiplied by."""
+    return 0.1 * math.log(float(scaling["factor"])) + 1.0 if scaling and scaling.get("kind") == "yarn" else 1.0
+
+
 @POSITIONS.register("rotary")
 class Rotary(Part):
-    """params: head_dim, theta, scaling (None or the llama3 dict), max_positions, dims (how many dimensions of a head are
+    """params: head_dim, theta, scaling (None, the llama3 dict or the YaRN one: "kind" "yarn", factor, original, fast,
+    slow), max_positions, dims (how many dimensions of a head are
     turned, at frequencies theta^(-2i/dims); default head_dim).  With dims < head_dim the tables still have head_dim / 2
     columns, the ones behind dims / 2 at angle zero (`head_order` says which dimensions a mixer puts there)."""
 
@@ -58,6 +82,7 @@ class Rotary(Part):
             raise ValueError(f"rotary: {self.dims} turned dimensions must be even and at most head_dim {self.head_dim}")
         self.max_positions = int(self._need("max_positions"))
         self.inv_freq = rotary_inv_freq(self.dims, float(self._need("theta")), self.params.get("scaling"))
+        self.magnitude = rotary_magnitude(self.params.get("scaling"))
         self.cos = self.sin = None
 
     def tables(self):
@@ -66,8 +91,8 @@ class Rotary(Part):
             pos = torch.arange(self.max_positions, dtype=torch.float64)
             freq = torch.cat([self.inv_freq, torch.zeros((self.head_dim - self.dims) // 2, dtype=torch.float64)])
             ang = pos[:, None] * freq[None, :]
-            self.cos = torch.cos(ang).to(torch.float32).to(self.rt.device).contiguous()
-            self.sin = torch.sin(ang).to(torch.float32).to(self.rt.device).contiguous()
+            self.cos = (torch.cos(ang) * self.magnitude).to(torch.float32).to(self.rt.device).contiguous()
+            self.sin = (torch.sin(ang) * self.magnitude).to(torch.float32).to(self.rt.device).contiguous()
         return self.cos, self.sin
 
     def head_order(self) -> list | None:
@@ -77,6 +102,8 @@ class Rotary(Part):
         the dimensions, so a query and a key that are both kept in this order score as before."""
         if self.dims == self.head_dim:
             return None
+        if self.magnitude != 1.0:
+            raise ValueError("rotary: dimensions at angle zero would take the scaling's magnitude")
         r, half = self.dims // 2, self.head_dim // 2
         rest = list(range(self.dims, self.head_dim))
         return list(range(r)) + rest[:half - r] + list(range(r, self.dims)) + rest[half - r:]
