@@ -6,7 +6,7 @@
     python bench.py --shape 8b --workload baseline      # 32 prompts of 128..4,096 tokens, 256 steps
     python bench.py --profile [--batch 64]              # device time per kind of kernel, on standard error
     python bench.py --impl reference --steps K          # the reference's own benchmark program (CPU)
-    python bench.py --design fuvipel|fovirax|pusunex|bogupel|goridra [--beside llama,fovirax] [--widths 1024,2048,3072] [--profile]
+    python bench.py --design fuvipel|fovirax|pusunex|bogupel|goridra|mavinex [--beside llama,fovirax] [--widths 1024,2048,3072] [--profile]
                                                         # that design beside a Llama of equal width and depth
 
 Prints ONE JSON line.  `value` is decoded tokens per second at the given batch (default
@@ -455,6 +455,30 @@ def goridra_shape(width: int, layers: int, vocab: int) -> dict:
                        {"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": 4 * width}} for i in range(layers)]}
 
 
+def mavinex_shape(width: int, layers: int, vocab: int) -> dict:
+    """A Mavinex of real layer sizes: layers of an attention (heads of 128, four query heads to a key head, a window of
+    1,024 keys, all of each head turned, frequencies rescaled by wavelength) beside a selective scan over 2 x width channels
+    with 16 states each (step sizes through a rank of width / 16, four taps), in turn with layers of attention over a latent
+    of 192 and a turned key part of 64 (the same window, a sink and a gate per head); on every layer a mixture of 8 experts
+    of 2/3 x width, two chosen.  No shared weights: as many distinct layers as runs."""
+    heads = width // 128
+    ff = (2 * width // 3 + 63) // 64 * 64
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": 8, "top": 2}}
+    par = {"type": "parallel", "mlp": moe,
+           "mixer": {"left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                              "mask": {"size": 1024},
+                              "rot": {"dims": 128, "base": 500000.0,
+                                      "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+                     "right": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}}}
+    lat = {"type": "latent_attention", "mlp": moe,
+           "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 192, "scale": 192 ** -0.5,
+                     "mask": {"size": 1024},
+                     "rot": {"dims": 64, "base": 10000.0,
+                             "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    return {"architecture": "Mavinex", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+            "postln_alpha": 2.0, "layers": [lat if i % 2 else par for i in range(layers)]}
+
+
 def llama_shape(width: int, layers: int, vocab: int) -> dict:
     """The Llama decoder of the same width, depth and vocabulary: heads of 128, four query heads to a key head,
     a SwiGLU of 8/3 x width (the same weights as a two-matrix feed-forward of 4 x width)."""
@@ -474,6 +498,7 @@ def design_compare(args) -> int:
     from oracle_engine_b200.config.fovirax import FoviraxConfig
     from oracle_engine_b200.config.fuvipel import FuvipelConfig
     from oracle_engine_b200.config.goridra import GoridraConfig
+    from oracle_engine_b200.config.mavinex import MavinexConfig
     from oracle_engine_b200.config.pusunex import PusunexConfig
     from oracle_engine_b200.engine.engine import Engine
     designs = {"fuvipel": lambda *a: FuvipelConfig.from_dict(fuvipel_shape(*a)),
@@ -481,6 +506,7 @@ def design_compare(args) -> int:
                "pusunex": lambda *a: PusunexConfig.from_dict(pusunex_shape(*a)),
                "bogupel": lambda *a: BogupelConfig.from_dict(bogupel_shape(*a)),
                "goridra": lambda *a: GoridraConfig.from_dict(goridra_shape(*a)),
+               "mavinex": lambda *a: MavinexConfig.from_dict(mavinex_shape(*a)),
                "llama": lambda *a: LlamaConfig.from_dict(llama_shape(*a))}
     beside = [b for b in (args.beside or "llama").split(",") if b and b != args.design]
     unknown = [b for b in beside if b not in designs]
@@ -644,7 +670,7 @@ def main():
     ap.add_argument("--profile", action="store_true",
                     help="print device time per kind of kernel of a prompt step and a decode step on standard error, "
                          "and nothing else")
-    ap.add_argument("--design", default=None, choices=["fuvipel", "fovirax", "pusunex", "bogupel", "goridra"],
+    ap.add_argument("--design", default=None, choices=["fuvipel", "fovirax", "pusunex", "bogupel", "goridra", "mavinex"],
                     help="measure this design beside the Llama decoder at equal sizes instead of the headline workload")
     ap.add_argument("--beside", default=None, help="the designs to measure beside --design, comma-separated (default llama)")
     ap.add_argument("--widths", default="1024,2048,3072", help="model widths of --design")

@@ -456,9 +456,11 @@ template <typename T>
 int launch_scan(const ScanArgs<T>& a, int n_seqs, cudaStream_t st) {
     if (n_seqs <= 0) return 0;
     if (a.C < 1 || a.N < 1 || a.N > 256 || n_seqs > 65535) return OE_ERR_UNSUPPORTED;
-    // few channels and sequences: a channel's states over more lanes
+    // few channels and sequences: a channel's states over more lanes.  float32: the same lanes whatever the batch, so that
+    // the order of a read-out's sum is always the same
+    const long long pairs = (sizeof(T) == 4 ? 1LL : (long long)n_seqs) * a.C;
     int per = 4;
-    while (per < 16 && per < a.N && (lanes_for(a.N, per) > 32 || (long long)n_seqs * a.C * lanes_for(a.N, per) > BUSY_THREADS)) per *= 2;
+    while (per < 16 && per < a.N && (lanes_for(a.N, per) > 32 || pairs * lanes_for(a.N, per) > BUSY_THREADS)) per *= 2;
     const int L = lanes_for(a.N, per);
     const dim3 grid((a.C + THREADS / L - 1) / (THREADS / L), n_seqs);
 #define OE_SCAN(P, LL) if (per == P && L == LL) return oe_launch(selective_scan_kernel<T, P, LL, 0>, grid, dim3(THREADS), 0, st, a);

@@ -118,7 +118,8 @@ class SelectiveScan(Part):
         matmul_nt(self.rt, thin, u, self.w_x)
         y = buf("ssm.y", T, C)
         z, off_b, off_c = xz[:, C:2 * C], self.ldw, self.ldw + self.N
-        if ctx.all_decode and ctx.n_tokens == ctx.n_seqs:
+        # float32 serving makes the step sizes the one way, so that a position's logits are the same bits under every cut
+        if self.rt.dtype != f32 and ctx.all_decode and ctx.n_tokens == ctx.n_seqs:
             ops.selective_step(y, state["S"], u, self.w_dt, 0, self.rank, self.dt_bias, thin, off_b, off_c, self.A2, self.skip,
                                z, ctx)
         else:
