@@ -126,6 +126,84 @@ __device__ __forceinline__ void pair_columns(int i, int rot, int halves, int& fi
     else { first = 2 * i; second = 2 * i + 1; }
 }
 
+// bfloat16 rows in 16-byte pieces: dk, dv and rot multiples of 8, pairs interleaved, so that a piece holds four pairs of one
+// head or eight values that pass.  The row's pieces stay in registers between the sums and the turn.
+template <int KEEP>
+__global__ void __launch_bounds__(ROW_THREADS)
+qkv_row_norm_rot_write_vec_kernel(bf16* qkv, bf16* kcache, bf16* vcache, const RowPrepArgs a) {
+    __shared__ float red[2][32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int b = a.tok_seq[t];
+    if (b < 0) return;
+    const int pos = a.tok_pos[t];
+    const int page = a.tables[(size_t)b * a.max_pages + pos / OE_PAGE];
+    bf16* row = qkv + (size_t)t * a.ld;
+    const int qp = a.H * a.dk / 8, kp = a.G * a.dk / 8, vp = a.G * a.dv / 8;
+    uint4 keep[KEEP];
+    float s = 0.f, u = 0.f;
+#pragma unroll
+    for (int j = 0; j < KEEP; j++) {
+        const int e = threadIdx.x + j * ROW_THREADS;
+        keep[j] = make_uint4(0u, 0u, 0u, 0u);
+        if (e < qp + kp + vp) keep[j] = reinterpret_cast<const uint4*>(row)[e];
+        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&keep[j]);
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; i++) { const float2 f = __bfloat1622float2(p[i]); ss = fmaf(f.x, f.x, fmaf(f.y, f.y, ss)); }
+        if (e < qp) s += ss;
+        else if (e < qp + kp) u += ss;
+    }
+    float sq = 1.f, sk = 1.f;
+    if (a.qw) {
+        s = block_sum(s, red[0]);
+        u = block_sum(u, red[1]);
+        sq = 1.f / sqrtf(s / (float)(a.H * a.dk) + a.eps);
+        sk = 1.f / sqrtf(u / (float)(a.G * a.dk) + a.eps);
+    }
+    const float* cr = a.cos_t + (size_t)pos * (a.rot / 2);
+    const float* sr = a.sin_t + (size_t)pos * (a.rot / 2);
+#pragma unroll
+    for (int j = 0; j < KEEP; j++) {
+        const int e = threadIdx.x + j * ROW_THREADS;
+        if (e >= qp + kp + vp) continue;
+        if (e >= qp && page < 0) continue;
+        if (e >= qp + kp) {
+            const int c = (e - qp - kp) * 8, head = c / a.dv;
+            *reinterpret_cast<uint4*>(vcache + (((size_t)page * a.G + head) * OE_PAGE + (pos % OE_PAGE)) * a.dv + (c - head * a.dv)) = keep[j];
+            continue;
+        }
+        const bool key = e >= qp;
+        const int c = (key ? e - qp : e) * 8, head = c / a.dk, d = c - head * a.dk;
+        const float sc = key ? sk : sq;
+        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&keep[j]);
+        float v[8];
+#pragma unroll
+        for (int i = 0; i < 4; i++) { const float2 f = __bfloat1622float2(p[i]); v[2 * i] = f.x * sc; v[2 * i + 1] = f.y * sc; }
+        if (a.qw) {
+            const float4* w = reinterpret_cast<const float4*>((key ? a.kw : a.qw) + c);
+            const float4 w0 = w[0], w1 = w[1];
+            v[0] *= w0.x; v[1] *= w0.y; v[2] *= w0.z; v[3] *= w0.w; v[4] *= w1.x; v[5] *= w1.y; v[6] *= w1.z; v[7] *= w1.w;
+        }
+        if (d < a.rot) {
+            const float4 cs = *reinterpret_cast<const float4*>(cr + d / 2), sn = *reinterpret_cast<const float4*>(sr + d / 2);
+            const float cc[4] = {cs.x, cs.y, cs.z, cs.w}, ss[4] = {sn.x, sn.y, sn.z, sn.w};
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const float x = v[2 * i], y = v[2 * i + 1];
+                v[2 * i] = x * cc[i] - y * ss[i];
+                v[2 * i + 1] = y * cc[i] + x * ss[i];
+            }
+        }
+        __nv_bfloat162 o[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) o[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        bf16* dst = key ? kcache + (((size_t)page * a.G + head) * OE_PAGE + (pos % OE_PAGE)) * a.dk + d : row + c;
+        *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(o);
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS)
 qkv_row_norm_rot_write_kernel(T* qkv, T* kcache, T* vcache, const RowPrepArgs a) {
@@ -232,6 +310,16 @@ int launch_row_prep(T* qkv, long long ld, T* kcache, T* vcache, const float* qw,
     a.ld = ld; a.qw = qw; a.kw = kw; a.eps = eps; a.cos_t = cos_t; a.sin_t = sin_t; a.rot = rot; a.halves = halves;
     a.tables = tables; a.max_pages = max_pages; a.tok_seq = tok_seq; a.tok_pos = tok_pos;
     a.n_tokens = n_tokens; a.H = H; a.G = G; a.dk = dk; a.dv = dv;
+    if constexpr (sizeof(T) == 2) {
+        const bool vec = dk % 8 == 0 && dv % 8 == 0 && rot % 8 == 0 && (rot == 0 || !halves) && ld % 8 == 0 &&
+                         !(((uintptr_t)qkv | (uintptr_t)kcache | (uintptr_t)vcache | (uintptr_t)qw | (uintptr_t)kw | (uintptr_t)cos_t |
+                            (uintptr_t)sin_t) & 15);
+        const int pieces = (H * dk + G * dk + G * dv) / 8;
+        if (vec && pieces <= 2 * ROW_THREADS)
+            return oe_launch(qkv_row_norm_rot_write_vec_kernel<2>, dim3(n_tokens), dim3(ROW_THREADS), 0, st, qkv, kcache, vcache, a);
+        if (vec && pieces <= 8 * ROW_THREADS)
+            return oe_launch(qkv_row_norm_rot_write_vec_kernel<8>, dim3(n_tokens), dim3(ROW_THREADS), 0, st, qkv, kcache, vcache, a);
+    }
     return oe_launch(qkv_row_norm_rot_write_kernel<T>, dim3(n_tokens), dim3(ROW_THREADS), 0, st, qkv, kcache, vcache, a);
 }
 

@@ -811,16 +811,16 @@ def gdelta_scan(o: torch.Tensor, state: torch.Tensor, packed: torch.Tensor, v: t
 
 def causal_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, state: torch.Tensor,
                 ctx) -> None:
-    """out[t, c] = silu(sum_j w[c, j] x[t - (taps - 1) + j, c] + bias[c]) over each sequence's rows, the rows before the
+    """out[t, c] = silu(sum_j w[j, c] x[t - (taps - 1) + j, c] + bias[c]) over each sequence's rows, the rows before the
     step's first from state [slots, max(taps - 1, 1), C] (float32), which then receives the sequence's last taps - 1 rows.
-    out [T, C] contiguous and x [T, >= C] (row stride free) of one dtype; w float32 [C, taps], bias float32 [C] or None."""
+    out [T, C] contiguous and x [T, >= C] (row stride free) of one dtype; w float32 [taps, C], bias float32 [C] or None."""
     _dev(out, x, w, bias, state)
     T, C = out.shape
-    taps = w.shape[1]
+    taps = w.shape[0]
     for t, n in ((w, "w"), (state, "state")) + (((bias, "bias"),) if bias is not None else ()):
         _f32c(t, n)
     if x.dtype != out.dtype or out.dtype not in _SUFFIX or not out.is_contiguous() or x.stride(1) != 1 or x.shape[0] < T \
-            or x.shape[1] < C or w.shape[0] != C or tuple(state.shape[1:]) != (max(taps - 1, 1), C) \
+            or x.shape[1] < C or w.shape[1] != C or tuple(state.shape[1:]) != (max(taps - 1, 1), C) \
             or (bias is not None and bias.numel() != C):
         raise KernelError("causal_conv: shapes do not agree")
     one_each = bool(ctx.all_decode and ctx.n_tokens == ctx.n_seqs) and 2 <= taps <= 4

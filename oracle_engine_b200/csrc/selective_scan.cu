@@ -1,6 +1,6 @@
 // Selective scan: a recurrence with a state of N values per channel whose decay, input and read-out depend on the token.
 //
-//   causal_conv       out[t, c] = silu(sum_j w[c][j] x[t - (taps - 1) + j, c] + b[c]) per sequence: rows before a step's first
+//   causal_conv       out[t, c] = silu(sum_j w[j][c] x[t - (taps - 1) + j, c] + b[c]) per sequence: rows before a step's first
 //                     token come from the sequence's kept rows [taps - 1, C] (float32, zeros at its start).  In a step of
 //                     one token per sequence the same kernel shifts the kept rows.
 //   conv_rows_state   the kept rows after a step of any other kind.
@@ -11,13 +11,13 @@
 //
 // A channel's N states belong to L adjacent lanes, lane l keeping states l PER .. l PER + PER - 1 in registers for all
 // tokens of the step; b and c, which every channel reads, go through shared memory a few tokens at a time.  The decay is
-// exp2(dt * A2) with A2 = A log2(e) made once.  Without segments a step's tokens of one sequence are walked in order,
+// 2^(dt A2) with A2 = A log2(e) made once.  Without segments a step's tokens of one sequence are walked in order,
 // whatever their number: the cut of a sequence into steps changes no bit.
 //
 // A long prompt in segments (oe_selective_scan_segments): the recurrence is linear in the state, so a sequence's tokens are
 // cut into segments of seg_len that run side by side.  Pass 1 walks every segment but a sequence's last from a zero state
-// and keeps its end state L_g and the sum s_g of its step sizes (the product of a segment's decays is exp2(s_g A2));
-// selective_join_kernel makes every segment's true entering state, E_0 = S, E_(g+1) = exp2(s_g A2) E_g + L_g; pass 2
+// and keeps its end state L_g and the sum s_g of its step sizes (the product of a segment's decays is 2^(s_g A2));
+// selective_join_kernel makes every segment's true entering state, E_0 = S, E_(g+1) = 2^(s_g A2) E_g + L_g; pass 2
 // walks every segment from its E_g and writes the outputs, a sequence's last segment also the state.
 #include "common.cuh"
 
@@ -51,28 +51,53 @@ __device__ __forceinline__ void store_vec(T* p, const float (&o)[V]) {
     for (int i = 0; i < (BYTES + 15) / 16; i++) reinterpret_cast<uint4*>(p)[i] = reinterpret_cast<uint4*>(t)[i];
 }
 
-// grid (token tiles of `per`, channel tiles).  A thread owns V adjacent channels and walks `per` tokens of the packed
-// batch with the window of the last TAPS rows in registers; at a sequence's first token of the step the window is filled
-// from the kept rows.  `shift`: every sequence brings one token, its thread also moves the kept rows on.
-template <typename T, int TAPS, int V>
+// grid (token tiles of PT, channel tiles).  A thread owns V adjacent channels and takes the tile's tokens with the window of
+// the last TAPS rows in registers.  A tile inside one sequence, its first window included, asks for all its rows at once;
+// any other goes token by token and fills the window anew at a sequence's first token of the step, from the kept rows.
+// `shift`: every sequence brings one token, its thread also moves the kept rows on.  w [taps, C].
+template <typename T, int TAPS, int V, int PT>
 __global__ void __launch_bounds__(THREADS)
 causal_conv_kernel(T* out, const T* x, long long ldx, const float* __restrict__ w, const float* __restrict__ bias, float* state,
                    const int* __restrict__ tok_seq, const int* __restrict__ seq_slot, const int* __restrict__ cu_q,
-                   int n_tokens, int C, int per, int shift) {
+                   int n_tokens, int C, int shift) {
+    const int c = (blockIdx.y * THREADS + threadIdx.x) * V;
+    float k[TAPS][V], b[V];
+    if (c < C) {
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) load_vec<float, V>(k[j], w + (size_t)j * C + c);
+#pragma unroll
+        for (int i = 0; i < V; i++) b[i] = 0.f;
+        if (bias) load_vec<float, V>(b, bias + c);
+    }
     pdl_launch_dependents();
     pdl_wait();
-    const int c = (blockIdx.y * THREADS + threadIdx.x) * V;
     if (c >= C) return;
-    float k[TAPS][V], win[TAPS][V], b[V];
+    const int t0 = blockIdx.x * PT;
+    if (PT > 1 && t0 + PT <= n_tokens) {
+        const int s = tok_seq[t0];
+        if (s >= 0 && s == tok_seq[t0 + PT - 1] && t0 - cu_q[s] >= TAPS - 1) {
+            float rows[PT + TAPS - 1][V];
 #pragma unroll
-    for (int i = 0; i < V; i++) {
-        b[i] = bias ? bias[c + i] : 0.f;
+            for (int r = 0; r < PT + TAPS - 1; r++) load_vec<T, V>(rows[r], x + (size_t)(t0 - (TAPS - 1) + r) * ldx + c);
 #pragma unroll
-        for (int j = 0; j < TAPS; j++) k[j][i] = w[(size_t)(c + i) * TAPS + j];
+            for (int t = 0; t < PT; t++) {
+                float y[V];
+#pragma unroll
+                for (int i = 0; i < V; i++) {
+                    float a = b[i];
+#pragma unroll
+                    for (int j = 0; j < TAPS; j++) a = fmaf(k[j][i], rows[t + j][i], a);
+                    y[i] = silu_f(a);
+                }
+                store_vec<T, V>(out + (size_t)(t0 + t) * C + c, y);
+            }
+            return;
+        }
     }
-    const int t_end = min(n_tokens, (int)(blockIdx.x + 1) * per);
+    float win[TAPS][V];
+    const int t_end = min(n_tokens, t0 + PT);
     int prev_seq = -1;
-    for (int t = blockIdx.x * per; t < t_end; t++) {
+    for (int t = t0; t < t_end; t++) {
         const int s = tok_seq[t];
         if (s < 0) { prev_seq = -1; continue; }
         const int rel = t - cu_q[s];
@@ -123,7 +148,7 @@ causal_conv_any_kernel(T* out, const T* x, long long ldx, const float* __restric
     for (int j = 0; j < taps; j++) {
         const int r = rel - (taps - 1) + j;
         const float v = r >= 0 ? to_f32(x[(size_t)(t - rel + r) * ldx + c]) : st[(size_t)(rel + j) * C + c];
-        a = fmaf(w[(size_t)c * taps + j], v, a);
+        a = fmaf(w[(size_t)j * C + c], v, a);
     }
     out[(size_t)t * C + c] = from_f32<T>(silu_f(a));
 }
@@ -197,6 +222,13 @@ __device__ __forceinline__ void store_states(float* p, const float (&s)[PER], in
     for (int i = 0; i < PER; i++) if (first + i < N) p[first + i] = s[i];
 }
 
+// 2^x by the hardware's instruction; a result too small for a normal number is zero (a decay: the state is gone).
+__device__ __forceinline__ float decay_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 template <int L>
 __device__ __forceinline__ float lanes_sum(float v) {
 #pragma unroll
@@ -215,7 +247,7 @@ __device__ __forceinline__ float scan_token(float (&s)[PER], const float (&a2)[P
             const float4 b = *reinterpret_cast<const float4*>(sb + i);
             const float bb[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
-            for (int e = 0; e < 4; e++) s[(i + e) % PER] = fmaf(exp2f(dt * a2[(i + e) % PER]), s[(i + e) % PER], du * bb[e]);
+            for (int e = 0; e < 4; e++) s[(i + e) % PER] = fmaf(decay_exp2(dt * a2[(i + e) % PER]), s[(i + e) % PER], du * bb[e]);
             if (OUT) {
                 const float4 c = *reinterpret_cast<const float4*>(sc + i);
                 acc0 = fmaf(s[i], c.x, acc0); acc1 = fmaf(s[(i + 1) % PER], c.y, acc1);
@@ -225,7 +257,7 @@ __device__ __forceinline__ float scan_token(float (&s)[PER], const float (&a2)[P
     } else {
 #pragma unroll
         for (int i = 0; i < PER; i++) {
-            s[i] = fmaf(exp2f(dt * a2[i]), s[i], du * sb[i]);
+            s[i] = fmaf(decay_exp2(dt * a2[i]), s[i], du * sb[i]);
             if (OUT) acc0 = fmaf(s[i], sc[i], acc0);
         }
     }
@@ -329,7 +361,7 @@ selective_join_kernel(const float* state, float* seg_state, const float* seg_dt,
     float s = state[(long long)slot * CN + e];
     for (int g = 0; (g + 1) * seg_len < n; g++) {
         const size_t at = (size_t)b * n_seg + g;
-        s = fmaf(exp2f(seg_dt[at * C + c] * a2), s, seg_state[at * CN + e]);
+        s = fmaf(decay_exp2(seg_dt[at * C + c] * a2), s, seg_state[at * CN + e]);
         seg_state[at * CN + e] = s;
     }
 }
@@ -423,18 +455,19 @@ int launch_conv(T* out, const T* x, long long ldx, const float* w, const float* 
     }
     // 16-byte pieces where the rows allow it and there are enough tokens; few tokens: a thread per channel
     constexpr int V = 16 / (int)sizeof(T);
-    const bool vec = C % V == 0 && C % 4 == 0 && (ldx * (long long)sizeof(T)) % 16 == 0 &&
-                     !(((uintptr_t)out | (uintptr_t)x | (uintptr_t)state) & 15) && (long long)n_tokens * C >= (1LL << 18);
-    const int per = n_tokens >= 1024 ? 8 : 1;
+    constexpr int PT = 8;
+    const bool vec = C % V == 0 && C % 4 == 0 && (ldx * (long long)sizeof(T)) % 16 == 0 && !one_each &&
+                     !(((uintptr_t)out | (uintptr_t)x | (uintptr_t)state | (uintptr_t)w | (uintptr_t)bias) & 15) &&
+                     (long long)n_tokens * C >= (1LL << 20);
     const int width = THREADS * (vec ? V : 1);
-    const dim3 grid((n_tokens + per - 1) / per, (C + width - 1) / width);
+    const dim3 grid(vec ? (n_tokens + PT - 1) / PT : n_tokens, (C + width - 1) / width);
     if (grid.y > 65535) return OE_ERR_UNSUPPORTED;
 #define OE_CONV(TAPS)                                                                                                          \
     if (taps == TAPS) {                                                                                                        \
-        if (vec) return oe_launch(causal_conv_kernel<T, TAPS, V>, grid, dim3(THREADS), 0, st, out, x, ldx, w, bias, state, tok_seq,  \
-                                  seq_slot, cu_q, n_tokens, C, per, one_each);                                                 \
-        return oe_launch(causal_conv_kernel<T, TAPS, 1>, grid, dim3(THREADS), 0, st, out, x, ldx, w, bias, state, tok_seq, seq_slot, \
-                         cu_q, n_tokens, C, per, one_each);                                                                    \
+        if (vec) return oe_launch(causal_conv_kernel<T, TAPS, V, PT>, grid, dim3(THREADS), 0, st, out, x, ldx, w, bias, state, \
+                                  tok_seq, seq_slot, cu_q, n_tokens, C, one_each);                                             \
+        return oe_launch(causal_conv_kernel<T, TAPS, 1, 1>, grid, dim3(THREADS), 0, st, out, x, ldx, w, bias, state, tok_seq,  \
+                         seq_slot, cu_q, n_tokens, C, one_each);                                                               \
     }
     OE_CONV(2) OE_CONV(3) OE_CONV(4)
 #undef OE_CONV

@@ -65,7 +65,7 @@ class SelectiveScan(Part):
         wx = to(get(n["x"]))
         self.w_x = torch.cat([wx[:self.rank], wx.new_zeros(pad, self.C), wx[self.rank:]], 0).contiguous()
         self.w_dt = torch.nn.functional.pad(to(get(n["dt"])), (0, pad)).contiguous()
-        self.conv_w, self.conv_b = f32(get(n["conv"])), f32(get(n["conv_bias"]))
+        self.conv_w, self.conv_b = f32(get(n["conv"])).T.contiguous(), f32(get(n["conv_bias"]))
         self.dt_bias, self.skip = f32(get(n["dt_bias"])), f32(get(n["D"]))
         self.A2 = (-torch.exp(f32(get(n["A_log"])).double()) * math.log2(math.e)).float().contiguous()
 
