@@ -7,6 +7,7 @@
     python -m oracle_engine_b200.csrc.microbench norm --rows 2048 --width 3072
     python -m oracle_engine_b200.csrc.microbench rope --tokens 4096
     python -m oracle_engine_b200.csrc.microbench scan --kind delta --tokens 2048 --batch 1 [--heads 16 --dim 128]
+    python -m oracle_engine_b200.csrc.microbench scan --kind selective --tokens 2048 --channels 4096 --states 16
     python -m oracle_engine_b200.csrc.microbench scan --kind decay --tokens 1 --batch 64 --heads 32 --dim 64
 
 In the manner of the reference's benchmark/micro_gemm.cpp (:97-128 correctness against a
@@ -222,6 +223,9 @@ def run_scan(a):
         nbytes = (qkv.numel() + gb.numel() + o.numel() + 2 * state.numel()) * 4
         report(f"delta_rule_scan tokens={T} batch={B} heads={H} ({d} x {d})", us, nbytes, 6.0 * T * B * H * d * d, err)
         return
+    if a.kind == "selective":
+        run_selective(a, ctx, dev)
+        return
     if a.kind == "general":
         import math
         C, rank, c = H * d, a.rank, math.exp(-0.5)
@@ -271,6 +275,43 @@ def run_scan(a):
     report(f"decay_scan tokens={T} batch={B} heads={H} ({d} x {d})", us, nbytes, 4.0 * T * B * H * d * d, err)
 
 
+def run_selective(a, ctx, dev):
+    """The selective scan (csrc/selective_scan.cu): prompts in one walk or as segments, single tokens in one launch."""
+    from ..parts.selective_scan import segment_plan
+    T, B, C, N, bf = a.tokens, a.batch, a.channels, a.states, torch.bfloat16
+    rows = T * B
+    u, z = torch.randn(rows, C, device=dev).to(bf), torch.randn(rows, C, device=dev).to(bf)
+    zdt, thin = torch.randn(rows, C, device=dev), torch.randn(rows, a.rank + 2 * N, device=dev)
+    bias, skip = torch.randn(C, device=dev) - 3, torch.randn(C, device=dev)
+    A2 = -torch.exp(torch.randn(C, N, device=dev)) * 1.4427
+    state, y = torch.zeros(B, C, N, device=dev), torch.empty(rows, C, device=dev, dtype=bf)
+    ctx.n_tokens, ctx.max_qlen, ctx.all_decode = rows, T, T == 1
+    off_b, off_c = a.rank, a.rank + N
+    n = min(T, 64)
+    if T == 1:
+        w = torch.randn(C, a.rank, device=dev).to(bf) * 0.1
+        zdt = (thin[:, :a.rank] @ w.float().T).contiguous()
+        fn = lambda i: ops.selective_step(y, state, u, w, 0, a.rank, bias, thin, off_b, off_c, A2, skip, z, ctx)     # noqa: E731
+        what = "selective_step"
+    else:
+        seg = segment_plan(C, N, B, T) if a.segments < 0 else None if a.segments < 2 else (-(-T // a.segments), a.segments)
+        if seg is not None:
+            seg = seg + (torch.empty(B * seg[1], C * N, device=dev), torch.empty(B * seg[1], C, device=dev))
+        fn = lambda i: ops.selective_scan(y, state, u, zdt, bias, thin, off_b, off_c, A2, skip, z, ctx, segments=seg)    # noqa: E731
+        what = f"selective_scan segments={1 if seg is None else seg[1]}"
+    fn(0)
+    dt = torch.nn.functional.softplus(zdt[:n, 0].double() + bias[0].double())
+    S, err = torch.zeros(N, dtype=torch.float64, device=dev), 0.0
+    for t in range(n):
+        S = torch.exp2(dt[t] * A2[0].double()) * S + dt[t] * u[t, 0].double() * thin[t, off_b:off_b + N].double()
+        want = (S @ thin[t, off_c:].double() + skip[0].double() * u[t, 0].double()) * torch.nn.functional.silu(z[t, 0].double())
+        err = max(err, (y[t, 0].double() - want).abs().item())
+    us = timed(fn, a.iters, a.once)
+    nbytes = 2 * (u.numel() + z.numel() + y.numel()) + 4 * (thin.numel() + 2 * state.numel() + A2.numel()) + \
+        (2 * C * a.rank if T == 1 else 4 * zdt.numel())
+    report(f"{what} tokens={T} batch={B} channels={C} states={N}", us, nbytes, 6.0 * rows * C * N, err)
+
+
 def main(argv=None):
     ap = argparse.ArgumentParser(prog="microbench")
     sub = ap.add_subparsers(dest="what", required=True)
@@ -313,8 +354,11 @@ def main(argv=None):
     r.add_argument("--kv-heads", type=int, default=8)
     r.add_argument("--head-dim", type=int, default=128)
     sc = sub.add_parser("scan")
-    sc.add_argument("--kind", default="delta", choices=["delta", "decay", "general"])
+    sc.add_argument("--kind", default="delta", choices=["delta", "decay", "general", "selective"])
     sc.add_argument("--rank", type=int, default=64, help="general: the rank of the decay's two-matrix projection")
+    sc.add_argument("--channels", type=int, default=4096, help="selective: channels (with --states each; --rank of the step sizes)")
+    sc.add_argument("--states", type=int, default=16)
+    sc.add_argument("--segments", type=int, default=-1, help="selective: segments side by side (-1: the rule's, 1: one walk)")
     sc.add_argument("--tokens", type=int, default=2048)
     sc.add_argument("--batch", type=int, default=1)
     sc.add_argument("--heads", type=int, default=16)

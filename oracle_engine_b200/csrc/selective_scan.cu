@@ -9,7 +9,7 @@
 //                     y_c = (sum_n S[c, n] c_n + D_c u_c) * silu(z_c)                                  everything in float32
 //   selective_step    the same for one token per sequence, with the step sizes' product inside: zdt_c = sum_j W[c, j] r_j.
 //
-// A channel's N states belong to L adjacent lanes, lane l keeping states l PER .. l PER + PER - 1 in registers for all
+// A channel's N states belong to L adjacent lanes (which may own a second channel), lane l keeping states l PER .. l PER + PER - 1 in registers for all
 // tokens of the step; b and c, which every channel reads, go through shared memory a few tokens at a time.  The decay is
 // 2^(dt A2) with A2 = A log2(e) made once.  Without segments a step's tokens of one sequence are walked in order,
 // whatever their number: the cut of a sequence into steps changes no bit.
@@ -28,6 +28,12 @@ constexpr int CHUNK = 16;        // tokens whose b and c are staged at once
 constexpr int THREADS = 128;
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// The output gate: of a result that is rounded to bfloat16 by the hardware's exponential and division.
+template <typename T>
+__device__ __forceinline__ float gate_silu(float z) {
+    if (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-z));
+    return silu_f(z);
+}
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 template <typename T, int V>
@@ -197,29 +203,61 @@ struct ScanArgs {
     int seg_len; float* seg_state; float* seg_dt;      // segments: [n_seqs, n_seg, C, N] and [n_seqs, n_seg, C]
 };
 
+// Two neighbouring states in one register pair: sm_100 multiplies and adds such pairs in one instruction.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pair_of(float lo, float hi) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float2 parts_of(f32x2 v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ f32x2 pair_mul(f32x2 x, f32x2 y) {
+    f32x2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(x), "l"(y));
+    return r;
+}
+__device__ __forceinline__ f32x2 pair_fma(f32x2 x, f32x2 y, f32x2 z) {
+    f32x2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(x), "l"(y), "l"(z));
+    return r;
+}
+
+// PER (a multiple of 4) states from `first` on; zeros behind the N-th.
 template <int PER>
-__device__ __forceinline__ void load_states(float (&s)[PER], const float* p, int first, int N, bool vec) {
-    if (PER % 4 == 0 && vec) {
+__device__ __forceinline__ void load_states(f32x2 (&s)[PER / 2], const float* p, int first, int N, bool vec) {
 #pragma unroll
-        for (int i = 0; i < PER; i += 4) {
-            const float4 q = first + i < N ? *reinterpret_cast<const float4*>(p + first + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-            s[i] = q.x; s[(i + 1) % PER] = q.y; s[(i + 2) % PER] = q.z; s[(i + 3) % PER] = q.w;
+    for (int i = 0; i < PER; i += 4) {
+        float4 q = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (vec) {
+            if (first + i < N) q = *reinterpret_cast<const float4*>(p + first + i);
+        } else {
+            if (first + i < N) q.x = p[first + i];
+            if (first + i + 1 < N) q.y = p[first + i + 1];
+            if (first + i + 2 < N) q.z = p[first + i + 2];
+            if (first + i + 3 < N) q.w = p[first + i + 3];
         }
-        return;
+        s[i / 2] = pair_of(q.x, q.y);
+        s[i / 2 + 1] = pair_of(q.z, q.w);
     }
-#pragma unroll
-    for (int i = 0; i < PER; i++) s[i] = first + i < N ? p[first + i] : 0.f;
 }
 template <int PER>
-__device__ __forceinline__ void store_states(float* p, const float (&s)[PER], int first, int N, bool vec) {
-    if (PER % 4 == 0 && vec) {
+__device__ __forceinline__ void store_states(float* p, const f32x2 (&s)[PER / 2], int first, int N, bool vec) {
 #pragma unroll
-        for (int i = 0; i < PER; i += 4)
-            if (first + i < N) *reinterpret_cast<float4*>(p + first + i) = make_float4(s[i], s[(i + 1) % PER], s[(i + 2) % PER], s[(i + 3) % PER]);
-        return;
+    for (int i = 0; i < PER; i += 4) {
+        const float2 x = parts_of(s[i / 2]), y = parts_of(s[i / 2 + 1]);
+        if (vec) {
+            if (first + i < N) *reinterpret_cast<float4*>(p + first + i) = make_float4(x.x, x.y, y.x, y.y);
+        } else {
+            if (first + i < N) p[first + i] = x.x;
+            if (first + i + 1 < N) p[first + i + 1] = x.y;
+            if (first + i + 2 < N) p[first + i + 2] = y.x;
+            if (first + i + 3 < N) p[first + i + 3] = y.y;
+        }
     }
-#pragma unroll
-    for (int i = 0; i < PER; i++) if (first + i < N) p[first + i] = s[i];
 }
 
 // 2^x by the hardware's instruction; a result too small for a normal number is zero (a decay: the state is gone).
@@ -236,40 +274,64 @@ __device__ __forceinline__ float lanes_sum(float v) {
     return v;
 }
 
-// One token: the state moves on, the read-out's share of this lane's states comes back.  sb, sc: this lane's part of the
-// token's b and c, PER values each, padded with zeros.
-template <int PER, bool OUT>
-__device__ __forceinline__ float scan_token(float (&s)[PER], const float (&a2)[PER], float dt, float du, const float* sb, const float* sc) {
-    float acc0 = 0.f, acc1 = 0.f;
-    if (PER % 4 == 0) {
+// One token of NC channels: their states move on, acc receives the read-outs' shares of this lane's states.  sb, sc: this
+// lane's part of the token's b and c, PER values each, padded with zeros, read once for all NC channels.
+template <int NC, int PER, bool OUT>
+__device__ __forceinline__ void scan_token(f32x2 (&s)[NC][PER / 2], const f32x2 (&a2)[NC][PER / 2], const float (&dt)[NC],
+                                           const float (&du)[NC], const float* sb, const float* sc, float (&acc)[NC]) {
+    f32x2 sum[NC][2], dt2[NC], du2[NC];
 #pragma unroll
-        for (int i = 0; i < PER; i += 4) {
-            const float4 b = *reinterpret_cast<const float4*>(sb + i);
-            const float bb[4] = {b.x, b.y, b.z, b.w};
+    for (int k = 0; k < NC; k++) {
+        sum[k][0] = sum[k][1] = 0ull;
+        dt2[k] = pair_of(dt[k], dt[k]);
+        du2[k] = pair_of(du[k], du[k]);
+    }
 #pragma unroll
-            for (int e = 0; e < 4; e++) s[(i + e) % PER] = fmaf(decay_exp2(dt * a2[(i + e) % PER]), s[(i + e) % PER], du * bb[e]);
+    for (int i = 0; i < PER / 2; i += 2) {
+        const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(sb + 2 * i);
+        ulonglong2 c = make_ulonglong2(0ull, 0ull);
+        if (OUT) c = *reinterpret_cast<const ulonglong2*>(sc + 2 * i);
+#pragma unroll
+        for (int k = 0; k < NC; k++) {
+            const float2 x = parts_of(pair_mul(dt2[k], a2[k][i])), y = parts_of(pair_mul(dt2[k], a2[k][i + 1]));
+            s[k][i] = pair_fma(pair_of(decay_exp2(x.x), decay_exp2(x.y)), s[k][i], pair_mul(du2[k], b.x));
+            s[k][i + 1] = pair_fma(pair_of(decay_exp2(y.x), decay_exp2(y.y)), s[k][i + 1], pair_mul(du2[k], b.y));
             if (OUT) {
-                const float4 c = *reinterpret_cast<const float4*>(sc + i);
-                acc0 = fmaf(s[i], c.x, acc0); acc1 = fmaf(s[(i + 1) % PER], c.y, acc1);
-                acc0 = fmaf(s[(i + 2) % PER], c.z, acc0); acc1 = fmaf(s[(i + 3) % PER], c.w, acc1);
+                sum[k][0] = pair_fma(s[k][i], c.x, sum[k][0]);
+                sum[k][1] = pair_fma(s[k][i + 1], c.y, sum[k][1]);
             }
         }
-    } else {
-#pragma unroll
-        for (int i = 0; i < PER; i++) {
-            s[i] = fmaf(decay_exp2(dt * a2[i]), s[i], du * sb[i]);
-            if (OUT) acc0 = fmaf(s[i], sc[i], acc0);
-        }
     }
-    return acc0 + acc1;
+#pragma unroll
+    for (int k = 0; k < NC; k++) {
+        const float2 x = parts_of(sum[k][0]), y = parts_of(sum[k][1]);
+        acc[k] = (x.x + x.y) + (y.x + y.y);
+    }
 }
 
-// grid (channel tiles, sequences[, segments]).  MODE 0: one walk; 1 and 2: the two passes over segments.
-template <typename T, int PER, int L, int MODE>
-__global__ void __launch_bounds__(THREADS)
+template <typename T, int NC>
+__device__ __forceinline__ void load_channels(float (&o)[NC], const T* p) {
+    if constexpr (NC == 2 && sizeof(T) == 2) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+        o[0] = f.x;
+        o[1] = f.y;
+    } else if constexpr (NC == 2) {
+        const float2 f = *reinterpret_cast<const float2*>(p);
+        o[0] = f.x;
+        o[1] = f.y;
+    } else {
+        o[0] = to_f32(p[0]);
+    }
+}
+
+// grid (channel tiles, sequences[, segments]).  MODE 0: one walk; 1 and 2: the two passes over segments.  A group of L lanes
+// owns NC adjacent channels (NC 2: C and ldz even, rows aligned for pairs).
+template <typename T, int PER, int L, int MODE, int NC>
+__global__ void __launch_bounds__(THREADS, NC == 2 ? 4 : 1)
 selective_scan_kernel(const ScanArgs<T> a) {
-    constexpr int CPB = THREADS / L, NP = PER * L;          // channels per block, states padded
+    constexpr int CPB = THREADS / L * NC, NP = PER * L;     // channels per block, states padded
     constexpr bool OUT = MODE != 1;
+    constexpr int AHEAD = 4;                                // tokens whose channel values are asked for at once
     __shared__ __align__(16) float stage[2][CHUNK][NP];
     pdl_launch_dependents();
     pdl_wait();
@@ -287,22 +349,38 @@ selective_scan_kernel(const ScanArgs<T> a) {
         if (MODE == 1 && last) return;                      // nothing comes after it
         n = min(n, first + a.seg_len);
     }
-    const int l = threadIdx.x % L, c = blockIdx.x * CPB + threadIdx.x / L;
+    const int l = threadIdx.x % L, c = blockIdx.x * CPB + threadIdx.x / L * NC;
     const bool mine = c < a.C;
-    const int cc = mine ? c : a.C - 1;
+    const int cc = mine ? c : a.C - NC;
     const bool vec = a.N % 4 == 0;
-    float* S = a.state + ((size_t)slot * a.C + cc) * a.N;
-    float s[PER], a2[PER];
-    load_states<PER>(a2, a.A2 + (size_t)cc * a.N, l * PER, a.N, vec);
-    if (MODE == 1) {
+    f32x2 s[NC][PER / 2], a2[NC][PER / 2];
+    float bias[NC], dw[NC], dt_sum[NC];
 #pragma unroll
-        for (int i = 0; i < PER; i++) s[i] = 0.f;
-    } else {
-        const float* enter = MODE == 2 && g > 0 ? a.seg_state + (((size_t)b * n_seg + g - 1) * a.C + cc) * a.N : S;
-        load_states<PER>(s, enter, l * PER, a.N, vec);
+    for (int k = 0; k < NC; k++) {
+        load_states<PER>(a2[k], a.A2 + (size_t)(cc + k) * a.N, l * PER, a.N, vec);
+        const float* enter = MODE == 2 && g > 0 ? a.seg_state + (((size_t)b * n_seg + g - 1) * a.C + cc + k) * a.N
+                                                : a.state + ((size_t)slot * a.C + cc + k) * a.N;
+        if (MODE == 1) {
+#pragma unroll
+            for (int i = 0; i < PER / 2; i++) s[k][i] = 0ull;
+        } else {
+            load_states<PER>(s[k], enter, l * PER, a.N, vec);
+        }
+        bias[k] = a.dt_bias[cc + k];
+        dw[k] = a.Dw[cc + k];
+        dt_sum[k] = 0.f;
     }
-    const float bias = a.dt_bias[cc], dw = a.Dw[cc];
-    float dt_sum = 0.f;
+    float dt[AHEAD][NC], u[AHEAD][NC], z[AHEAD][NC];
+    auto fetch = [&](int t0) {                              // tokens t0 .. t0 + AHEAD - 1 of the sequence (clamped to n - 1)
+#pragma unroll
+        for (int k = 0; k < AHEAD; k++) {
+            const size_t row = (size_t)(row0 + min(t0 + k, n - 1));
+            load_channels<float, NC>(dt[k], a.zdt + row * a.C + cc);
+            load_channels<T, NC>(u[k], a.u + row * a.C + cc);
+            if (OUT) load_channels<T, NC>(z[k], a.z + row * a.ldz + cc);
+        }
+    };
+    fetch(first);
     for (int c0 = first; c0 < n; c0 += CHUNK) {
         const int cn = min(CHUNK, n - c0);
         __syncthreads();
@@ -313,37 +391,54 @@ selective_scan_kernel(const ScanArgs<T> a) {
             if (OUT) stage[1][tt][i] = i < a.N ? row[a.off_c + i] : 0.f;
         }
         __syncthreads();
-        for (int t4 = 0; t4 < cn; t4 += 4) {
-            float dt[4], u[4], z[4];
+        for (int t4 = 0; t4 < cn; t4 += AHEAD) {
+            // what does not depend on the state comes first, for all of these tokens
+            float d_all[AHEAD][NC], u_now[AHEAD][NC], gate[AHEAD][NC];
 #pragma unroll
-            for (int k = 0; k < 4; k++) {
-                const size_t row = (size_t)(row0 + c0 + min(t4 + k, cn - 1));
-                dt[k] = a.zdt[row * a.C + cc];
-                u[k] = to_f32(a.u[row * a.C + cc]);
-                z[k] = OUT ? to_f32(a.z[row * a.ldz + cc]) : 0.f;
-            }
+            for (int k = 0; k < AHEAD; k++)
 #pragma unroll
-            for (int k = 0; k < 4; k++) {
+                for (int e = 0; e < NC; e++) {
+                    d_all[k][e] = softplus_f(dt[k][e] + bias[e]);
+                    u_now[k][e] = u[k][e];
+                    if (OUT) gate[k][e] = gate_silu<T>(z[k][e]);
+                }
+            if (c0 + t4 + AHEAD < n) fetch(c0 + t4 + AHEAD);
+#pragma unroll
+            for (int k = 0; k < AHEAD; k++) {
                 if (t4 + k < cn) {
-                    const float d = softplus_f(dt[k] + bias);
-                    if (MODE == 1) dt_sum += d;
-                    float y = scan_token<PER, OUT>(s, a2, d, d * u[k], &stage[0][t4 + k][l * PER], &stage[1][t4 + k][l * PER]);
+                    float d[NC], du[NC], y[NC];
+#pragma unroll
+                    for (int e = 0; e < NC; e++) {
+                        d[e] = d_all[k][e];
+                        du[e] = d[e] * u_now[k][e];
+                        if (MODE == 1) dt_sum[e] += d[e];
+                    }
+                    scan_token<NC, PER, OUT>(s, a2, d, du, &stage[0][t4 + k][l * PER], &stage[1][t4 + k][l * PER], y);
                     if (OUT) {
-                        y = lanes_sum<L>(y);
-                        if (mine && l == 0)
-                            a.y[(size_t)(row0 + c0 + t4 + k) * a.C + c] = from_f32<T>(fmaf(dw, u[k], y) * silu_f(z[k]));
+#pragma unroll
+                        for (int e = 0; e < NC; e++) y[e] = fmaf(dw[e], u_now[k][e], lanes_sum<L>(y[e])) * gate[k][e];
+                        T* dst = a.y + (size_t)(row0 + c0 + t4 + k) * a.C + c;
+                        if (mine && l == 0) {
+                            if constexpr (NC == 2 && sizeof(T) == 2) *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(y[0], y[1]);
+                            else
+#pragma unroll
+                                for (int e = 0; e < NC; e++) dst[e] = from_f32<T>(y[e]);
+                        }
                     }
                 }
             }
         }
     }
     if (!mine) return;
-    if (MODE == 1) {
-        store_states<PER>(a.seg_state + (((size_t)b * n_seg + g) * a.C + c) * a.N, s, l * PER, a.N, vec);
-        if (l == 0) a.seg_dt[((size_t)b * n_seg + g) * a.C + c] = dt_sum;
-        return;
+#pragma unroll
+    for (int k = 0; k < NC; k++) {
+        if (MODE == 1) {
+            store_states<PER>(a.seg_state + (((size_t)b * n_seg + g) * a.C + c + k) * a.N, s[k], l * PER, a.N, vec);
+            if (l == 0) a.seg_dt[((size_t)b * n_seg + g) * a.C + c + k] = dt_sum[k];
+        } else if (last) {
+            store_states<PER>(a.state + ((size_t)slot * a.C + c + k) * a.N, s[k], l * PER, a.N, vec);
+        }
     }
-    if (last) store_states<PER>(S, s, l * PER, a.N, vec);
 }
 
 // seg_state[b][g] becomes what segment g + 1 starts from.  One thread per (channel, state); grid (blocks, sequences).
@@ -388,13 +483,14 @@ selective_step_kernel(const ScanArgs<T> a, const T* __restrict__ W, int ldw, int
         row[k] = b < n_seqs ? a.cu_q[b] : 0;
         if (slot[k] >= 0 && a.cu_q[b + 1] <= row[k]) slot[k] = -1;
     }
-    float s[SG][PER], a2[PER], u[SG], z[SG];
-    load_states<PER>(a2, a.A2 + (size_t)cc * a.N, l * PER, a.N, vec);
+    f32x2 s[SG][1][PER / 2], a2[1][PER / 2];
+    float u[SG], z[SG];
+    load_states<PER>(a2[0], a.A2 + (size_t)cc * a.N, l * PER, a.N, vec);
 #pragma unroll
     for (int k = 0; k < SG; k++) {
         u[k] = z[k] = 0.f;
         if (slot[k] < 0) continue;
-        load_states<PER>(s[k], a.state + ((size_t)slot[k] * a.C + cc) * a.N, l * PER, a.N, vec);
+        load_states<PER>(s[k][0], a.state + ((size_t)slot[k] * a.C + cc) * a.N, l * PER, a.N, vec);
         u[k] = to_f32(a.u[(size_t)row[k] * a.C + cc]);
         z[k] = to_f32(a.z[(size_t)row[k] * a.ldz + cc]);
         const float* tr = a.thin + (size_t)row[k] * a.ldthin;
@@ -429,10 +525,13 @@ selective_step_kernel(const ScanArgs<T> a, const T* __restrict__ W, int ldw, int
         if (slot[k] < 0) continue;                          // the same for the whole block
         const float dt = softplus_f(lanes_sum<L>(zd[k]) + bias);
         const float* st = staged + k * per_seq + ldw + l * PER;
-        const float y = lanes_sum<L>(scan_token<PER, true>(s[k], a2, dt, dt * u[k], st, st + NP));
+        const float d[1] = {dt}, du[1] = {dt * u[k]};
+        float y[1];
+        scan_token<1, PER, true>(s[k], a2, d, du, st, st + NP, y);
+        y[0] = lanes_sum<L>(y[0]);
         if (!mine) continue;
-        if (l == 0) a.y[(size_t)row[k] * a.C + c] = from_f32<T>(fmaf(dw, u[k], y) * silu_f(z[k]));
-        store_states<PER>(a.state + ((size_t)slot[k] * a.C + c) * a.N, s[k], l * PER, a.N, vec);
+        if (l == 0) a.y[(size_t)row[k] * a.C + c] = from_f32<T>(fmaf(dw, u[k], y[0]) * gate_silu<T>(z[k]));
+        store_states<PER>(a.state + ((size_t)slot[k] * a.C + c) * a.N, s[k][0], l * PER, a.N, vec);
     }
 }
 
@@ -496,7 +595,7 @@ int launch_scan(const ScanArgs<T>& a, int n_seqs, cudaStream_t st) {
     while (per < 16 && per < a.N && (lanes_for(a.N, per) > 32 || pairs * lanes_for(a.N, per) > BUSY_THREADS)) per *= 2;
     const int L = lanes_for(a.N, per);
     const dim3 grid((a.C + THREADS / L - 1) / (THREADS / L), n_seqs);
-#define OE_SCAN(P, LL) if (per == P && L == LL) return oe_launch(selective_scan_kernel<T, P, LL, 0>, grid, dim3(THREADS), 0, st, a);
+#define OE_SCAN(P, LL) if (per == P && L == LL) return oe_launch(selective_scan_kernel<T, P, LL, 0, 1>, grid, dim3(THREADS), 0, st, a);
     OE_SCAN(4, 1) OE_SCAN(4, 2) OE_SCAN(4, 4) OE_SCAN(4, 8) OE_SCAN(4, 16) OE_SCAN(4, 32)
     OE_SCAN(8, 1) OE_SCAN(8, 2) OE_SCAN(8, 4) OE_SCAN(8, 8) OE_SCAN(8, 16) OE_SCAN(8, 32)
     OE_SCAN(16, 1) OE_SCAN(16, 2) OE_SCAN(16, 4) OE_SCAN(16, 8) OE_SCAN(16, 16)
@@ -512,16 +611,21 @@ int launch_segments(const ScanArgs<bf16>& a, int n_seqs, int n_seg, cudaStream_t
     int per = 8;
     while (per < 16 && per < a.N && (lanes_for(a.N, per) > 32 || (long long)n_seqs * n_seg * a.C * lanes_for(a.N, per) > BUSY_THREADS)) per *= 2;
     const int L = lanes_for(a.N, per);
-    const dim3 grid((a.C + THREADS / L - 1) / (THREADS / L), n_seqs, n_seg);
+    // two channels a lane, so that what is read of b and c serves both
+    const bool two = a.C % 2 == 0 && a.ldz % 2 == 0 && !(((uintptr_t)a.u | (uintptr_t)a.z | (uintptr_t)a.y) & 3) && !((uintptr_t)a.zdt & 7);
+    const int cpb = THREADS / L * (two ? 2 : 1);
+    const dim3 grid((a.C + cpb - 1) / cpb, n_seqs, n_seg);
     const long long blocks = ((long long)a.C * a.N + 255) / 256;
 #define OE_SCAN(P, LL)                                                                                                         \
     if (per == P && L == LL) {                                                                                                 \
-        int rc = oe_launch(selective_scan_kernel<bf16, P, LL, 1>, grid, dim3(THREADS), 0, st, a);                              \
+        int rc = two ? oe_launch(selective_scan_kernel<bf16, P, LL, 1, 2>, grid, dim3(THREADS), 0, st, a)                      \
+                     : oe_launch(selective_scan_kernel<bf16, P, LL, 1, 1>, grid, dim3(THREADS), 0, st, a);                     \
         if (rc) return rc;                                                                                                     \
         rc = oe_launch(selective_join_kernel, dim3((unsigned)blocks, n_seqs), dim3(256), 0, st, (const float*)a.state, a.seg_state, \
                        (const float*)a.seg_dt, a.A2, a.seq_slot, a.cu_q, a.C, a.N, a.seg_len, n_seg);                          \
         if (rc) return rc;                                                                                                     \
-        return oe_launch(selective_scan_kernel<bf16, P, LL, 2>, grid, dim3(THREADS), 0, st, a);                                \
+        if (two) return oe_launch(selective_scan_kernel<bf16, P, LL, 2, 2>, grid, dim3(THREADS), 0, st, a);                    \
+        return oe_launch(selective_scan_kernel<bf16, P, LL, 2, 1>, grid, dim3(THREADS), 0, st, a);                             \
     }
     OE_SCAN(8, 1) OE_SCAN(8, 2) OE_SCAN(8, 4) OE_SCAN(8, 8) OE_SCAN(8, 16) OE_SCAN(8, 32)
     OE_SCAN(16, 1) OE_SCAN(16, 2) OE_SCAN(16, 4) OE_SCAN(16, 8) OE_SCAN(16, 16)

@@ -31,6 +31,15 @@ SEGMENT_MIN = 32            # tokens of the shortest segment
 SEGMENT_THREADS = 148 * 1024     # threads of the scan that keep the GPU busy
 
 
+def segment_plan(C: int, N: int, n_seqs: int, longest: int) -> tuple | None:
+    """(tokens of a segment, segments a sequence) for a step whose longest sequence brings `longest` tokens, or None."""
+    lanes = -(-N // 16)
+    n_seg = max(1, min(-(-SEGMENT_THREADS // (C * lanes * max(1, n_seqs))), longest // SEGMENT_MIN))
+    seg_len = -(-(-(-longest // n_seg)) // 8) * 8
+    n_seg = -(-longest // seg_len)
+    return None if n_seg < 2 else (seg_len, n_seg)
+
+
 @MIXERS.register("selective_scan")
 class SelectiveScan(Part):
     graph_safe = True
@@ -94,12 +103,10 @@ class SelectiveScan(Part):
         longest = int(ctx.max_qlen)
         if self.rt.dtype != torch.bfloat16 or longest < SEGMENTS_FROM or torch.cuda.is_current_stream_capturing():
             return None             # (a captured step's longest sequence is a bound, not a length)
-        lanes = -(-self.N // 16)
-        n_seg = max(1, min(-(-SEGMENT_THREADS // (self.C * lanes * max(1, ctx.n_seqs))), longest // SEGMENT_MIN))
-        seg_len = -(-(-(-longest // n_seg)) // 8) * 8
-        n_seg = -(-longest // seg_len)
-        if n_seg < 2:
+        plan = segment_plan(self.C, self.N, ctx.n_seqs, longest)
+        if plan is None:
             return None
+        seg_len, n_seg = plan
         seg_state = self.rt.buffer("ssm.seg_state", ctx.n_seqs * n_seg, self.C * self.N, dtype=torch.float32)
         seg_dt = self.rt.buffer("ssm.seg_dt", ctx.n_seqs * n_seg, self.C, dtype=torch.float32)
         return seg_len, n_seg, seg_state, seg_dt
