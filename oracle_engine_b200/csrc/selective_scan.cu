@@ -28,7 +28,7 @@ constexpr int CHUNK = 16;        // tokens whose b and c are staged at once
 constexpr int THREADS = 128;
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
-// The output gate: of a result that is rounded to bfloat16 by the hardware's exponential and division.
+// silu of a result that is rounded to bfloat16 by the hardware's exponential and division.
 template <typename T>
 __device__ __forceinline__ float gate_silu(float z) {
     if (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-z));
@@ -36,25 +36,39 @@ __device__ __forceinline__ float gate_silu(float z) {
 }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
+// V consecutive values in pieces of 16 (or once 8) bytes; one value as it is.
 template <typename T, int V>
 __device__ __forceinline__ void load_vec(float (&o)[V], const T* p) {
-    if (V == 1) { o[0] = to_f32(p[0]); return; }
-    constexpr int BYTES = V * (int)sizeof(T);
-    __align__(16) T t[V];
+    if constexpr (V == 1) {
+        o[0] = to_f32(p[0]);
+    } else {
+        __align__(16) T t[V];
+        if constexpr (V * sizeof(T) == 8) {
+            *reinterpret_cast<uint2*>(t) = *reinterpret_cast<const uint2*>(p);
+        } else {
+            static_assert(V * sizeof(T) % 16 == 0, "pieces of 16 bytes");
 #pragma unroll
-    for (int i = 0; i < (BYTES + 15) / 16; i++) reinterpret_cast<uint4*>(t)[i] = reinterpret_cast<const uint4*>(p)[i];
+            for (int i = 0; i < V * (int)sizeof(T) / 16; i++) reinterpret_cast<uint4*>(t)[i] = reinterpret_cast<const uint4*>(p)[i];
+        }
 #pragma unroll
-    for (int i = 0; i < V; i++) o[i] = to_f32(t[i]);
+        for (int i = 0; i < V; i++) o[i] = to_f32(t[i]);
+    }
 }
 template <typename T, int V>
 __device__ __forceinline__ void store_vec(T* p, const float (&o)[V]) {
-    if (V == 1) { p[0] = from_f32<T>(o[0]); return; }
-    constexpr int BYTES = V * (int)sizeof(T);
-    __align__(16) T t[V];
+    if constexpr (V == 1) {
+        p[0] = from_f32<T>(o[0]);
+    } else {
+        __align__(16) T t[V];
 #pragma unroll
-    for (int i = 0; i < V; i++) t[i] = from_f32<T>(o[i]);
+        for (int i = 0; i < V; i++) t[i] = from_f32<T>(o[i]);
+        if constexpr (V * sizeof(T) == 8) {
+            *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(t);
+        } else {
 #pragma unroll
-    for (int i = 0; i < (BYTES + 15) / 16; i++) reinterpret_cast<uint4*>(p)[i] = reinterpret_cast<uint4*>(t)[i];
+            for (int i = 0; i < V * (int)sizeof(T) / 16; i++) reinterpret_cast<uint4*>(p)[i] = reinterpret_cast<uint4*>(t)[i];
+        }
+    }
 }
 
 // grid (token tiles of PT, channel tiles).  A thread owns V adjacent channels and takes the tile's tokens with the window of
@@ -93,7 +107,7 @@ causal_conv_kernel(T* out, const T* x, long long ldx, const float* __restrict__ 
                     float a = b[i];
 #pragma unroll
                     for (int j = 0; j < TAPS; j++) a = fmaf(k[j][i], rows[t + j][i], a);
-                    y[i] = silu_f(a);
+                    y[i] = gate_silu<T>(a);
                 }
                 store_vec<T, V>(out + (size_t)(t0 + t) * C + c, y);
             }
@@ -128,7 +142,7 @@ causal_conv_kernel(T* out, const T* x, long long ldx, const float* __restrict__ 
             float a = b[i];
 #pragma unroll
             for (int j = 0; j < TAPS; j++) a = fmaf(k[j][i], win[j][i], a);
-            y[i] = silu_f(a);
+            y[i] = gate_silu<T>(a);
         }
         store_vec<T, V>(out + (size_t)t * C + c, y);
         if (shift)
@@ -156,7 +170,7 @@ causal_conv_any_kernel(T* out, const T* x, long long ldx, const float* __restric
         const float v = r >= 0 ? to_f32(x[(size_t)(t - rel + r) * ldx + c]) : st[(size_t)(rel + j) * C + c];
         a = fmaf(w[(size_t)j * C + c], v, a);
     }
-    out[(size_t)t * C + c] = from_f32<T>(silu_f(a));
+    out[(size_t)t * C + c] = from_f32<T>(gate_silu<T>(a));
 }
 
 // grid (sequences, channel tiles); a thread owns a channel, so it reads its old rows before it writes them.
@@ -552,10 +566,10 @@ int launch_conv(T* out, const T* x, long long ldx, const float* w, const float* 
         if (grid.y > 65535) return OE_ERR_UNSUPPORTED;
         return oe_launch(causal_conv_any_kernel<T>, grid, dim3(THREADS), 0, st, out, x, ldx, w, bias, taps, (const float*)state, tok_seq, seq_slot, cu_q, C);
     }
-    // 16-byte pieces where the rows allow it and there are enough tokens; few tokens: a thread per channel
-    constexpr int V = 16 / (int)sizeof(T);
+    // four channels a thread where the rows allow it and there are enough tokens; few tokens: a thread per channel
+    constexpr int V = 4;
     constexpr int PT = 8;
-    const bool vec = C % V == 0 && C % 4 == 0 && (ldx * (long long)sizeof(T)) % 16 == 0 && !one_each &&
+    const bool vec = C % V == 0 && ldx % V == 0 && !one_each &&
                      !(((uintptr_t)out | (uintptr_t)x | (uintptr_t)state | (uintptr_t)w | (uintptr_t)bias) & 15) &&
                      (long long)n_tokens * C >= (1LL << 20);
     const int width = THREADS * (vec ? V : 1);

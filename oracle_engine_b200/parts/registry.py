@@ -32,13 +32,18 @@ Mixer  (MIXERS; e.g. attention)
 
     optional: parts with `joint_weight` (the attribute that holds the first matrix) whose forward takes `projected=`, a
     feed-forward also with `joint_epilogue(h, ctx)`, can have their first products computed as one by an arrangement
-    that gives both the same input (parts/block.py: JoinedInput)
+    that gives both the same input (parts/block.py: JoinedInput; parts/parallel.py for mixers side by side)
+
+    optional: a mixer made of mixers with output norms may hand those outputs over unnormed, with the norms' weights
+    (`normed_outputs`, `eps`); an arrangement that norms the sum then does all of it in one kernel
 
 FeedForward  (FEED_FORWARDS; dense or routed)
     forward(h, residual, ctx)            adds its output into residual
 
 Norm  (NORMS)
     forward(x) -> tensor                 x float32 [T, hidden] -> compute dtype
+    optional: add_into(dst, y, coef) adds the norm of a sublayer's output, sum_into(x, parts, alpha) replaces x by the norm
+    of alpha x plus a sublayer's output (parts/norms.py)
 
 PositionEncoding  (POSITIONS)            built once per model and name, shared by mixers
     tables(max_positions)                whatever its mixers read (e.g. cos/sin tables)
