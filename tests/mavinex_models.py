@@ -88,24 +88,24 @@ def random_config(rng):
             continue
         experts = rng.choice([1, 3, 5, 8, 12])
         mlp = None if rng.random() < 0.25 else moe(experts, rng.randint(1, min(4, experts)), rng.choice([32, 64, 50, 72]))
-        window = rng.choice([None, 1, 17, 64, 96, 136, 200])
-        base = rng.choice([10000.0, 250000.0, 500.0])
+        window = rng.choice([None, 1, 17, 64, 96, 140, 200])
+        base = rng.choice([10000.0, 300000.0, 500.0])
         if rng.random() < 0.5:
             heads = rng.choice([2, 4, 6, 8])
             kv = rng.choice([k for k in (1, 2, 4, 8) if heads % k == 0])
-            dim, vdim = rng.choice([32, 48, 64, 96, 40, 128]), rng.choice([32, 48, 80, 64, 24])
+            dim, vdim = rng.choice([32, 48, 64, 96, 40, 128]), rng.choice([32, 48, 96, 64, 24])
             dims = rng.choice([d for d in (0, 8, 16, 24, 32, dim) if d <= dim])
-            scaling = rng.choice([None, wave(rng.choice([2.0, 8.0]), 1.0, rng.choice([2.0, 4.0]), rng.choice([64, 512]))])
+            scaling = rng.choice([None, wave(rng.choice([2.0, 8.0]), 1.0, rng.choice([2.0, 4.0]), rng.choice([64, 700]))])
             layers.append(parallel(heads, kv, dim, vdim, dim ** -0.5, window, rot(dims, base, scaling) if dims else None,
                                    rng.choice([64, 128, 100, 256]), rng.choice([4, 8, 16, 32, 10]), rng.choice([3, 8, 12, 16]),
                                    rng.choice([2, 3, 4, 6]), mlp))
         else:
             rd = rng.choice([0, 8, 16, 32, 32])
-            scaling = rng.choice([None, yarn(rng.choice([2.0, 8.0]), rng.choice([128, 1024]), 32.0, 1.0)])
+            scaling = rng.choice([None, yarn(rng.choice([2.0, 8.0]), rng.choice([128, 2000]), 32.0, 1.0)])
             dim = rng.choice([16, 32, 64, 40])
             layers.append(latent(rng.choice([1, 2, 4, 5]), dim, rd, rng.choice([16, 32, 64, 24]), rng.choice([32, 64, 128, 50]),
                                  (dim + rd) ** -0.5, window, rot(rd, base, scaling) if rd else None, mlp))
-    return config(rng.choice([256, 448, 1000]), rng.choice([128, 192, 256, 320, 200]), rng.choice([1e-5, 1e-6]),
+    return config(rng.choice([256, 500, 1000]), rng.choice([128, 192, 256, 320, 200]), rng.choice([1e-5, 1e-6]),
                   rng.choice([0.8, 1.0, 2.5]), rng.choice([1.0, 12.0]), layers)
 
 

@@ -108,8 +108,8 @@ def test_model_description():
     assert m.layers[1].mixer.cache_bytes_per_query(100) == 24 * 80 * 4
 
 
-@pytest.mark.parametrize("rot", [mm.rot(16, 10000.0), mm.rot(48, 250000.0, mm.wave(8.0, 1.0, 4.0, 512)),
-                                 mm.rot(10, 1000.0, mm.wave(2.0, 1.0, 2.0, 40)), mm.rot(32, 10000.0, mm.yarn(8.0, 1024, 32.0, 1.0)),
+@pytest.mark.parametrize("rot", [mm.rot(16, 10000.0), mm.rot(40, 300000.0, mm.wave(6.0, 1.0, 5.0, 700)),
+                                 mm.rot(10, 1000.0, mm.wave(2.0, 1.0, 2.0, 40)), mm.rot(24, 20000.0, mm.yarn(6.0, 2000, 24.0, 2.0)),
                                  mm.rot(6, 50000.0, mm.yarn(40.0, 4096, 32.0, 1.0)), mm.rot(64, 10.0, mm.yarn(3.0, 9, 1.0, 1.0))])
 def test_rotary_tables_are_the_plain_models(rot):
     """Frequencies, both rescalings and the magnitude; a pair at position 0 is the magnitude and nothing else."""
